@@ -12,12 +12,13 @@
 //
 // Epilogues: bf16 output; fp32 output times alpha (the output head); SiLU(gate)*up for a
 // gate_up matrix whose rows are interleaved in blocks of 8 (8 gate rows, then the 8 up
-// rows of the same features), so that gate and up of a feature meet in one tile.
+// rows of the same features), so that gate and up of a feature meet in one tile; relu(x)^2 for a feed-forward without a gate.
 // The reference calls cublasGemmEx for every product (src/model/linear.cuh:8-37) and runs
 // the gated activation as a kernel of its own (src/model/activation.cuh:6-18).
 #include "common.cuh"
 
-enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU = 2, EPI_GELU = 3 };      // 2, 3: act(gate) * up with SiLU, with the tanh form of GELU
+// 2, 3: act(gate) * up with SiLU, with the tanh form of GELU; 4: relu(x)^2
+enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU = 2, EPI_GELU = 3, EPI_RELU2 = 4 };
 
 // 128-byte lines of each weight row a block asks L2 for at its start (and, under programmatic dependent
 // launch, before it waits for the kernel ahead of it).  Eight lines bring the first loads of the main loop
@@ -134,6 +135,10 @@ skinny_gemm_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, void*
             float sum = 0.f;
 #pragma unroll
             for (int w = 0; w < kSkinnyWarps; ++w) sum += red[w][row][tok];
+            if (EPI == EPI_RELU2) {
+                sum = fmaxf(sum, 0.f);
+                sum *= sum;
+            }
             if (EPI == EPI_F32) reinterpret_cast<float*>(out)[(int64_t)tok * N + n0 + row] = alpha * sum;
             else reinterpret_cast<bf16*>(out)[(int64_t)tok * N + n0 + row] = __float2bfloat16_rn(alpha * sum);
         }
@@ -155,6 +160,7 @@ static int launch_skinny(const void* W, const void* X, void* out, int M, int N, 
     if (epilogue == EPI_F32) return launch_skinny_epi<NT, EPI_F32>(W, X, out, M, N, K, alpha, stream);
     if (epilogue == EPI_SILU) return launch_skinny_epi<NT, EPI_SILU>(W, X, out, M, N, K, alpha, stream);
     if (epilogue == EPI_GELU) return launch_skinny_epi<NT, EPI_GELU>(W, X, out, M, N, K, alpha, stream);
+    if (epilogue == EPI_RELU2) return launch_skinny_epi<NT, EPI_RELU2>(W, X, out, M, N, K, alpha, stream);
     return CPM_BAD_ARGUMENT;
 }
 

@@ -13,8 +13,8 @@
 //
 // Epilogues: bf16 output, or SiLU(gate) * up for a gate_up weight whose rows are interleaved in
 // blocks of 8 (the 32 accumulator columns a thread reads at a time hold 8 gate, 8 up, 8 gate, 8
-// up values of 16 features), which saves the round trip of the [M, 2*inter] intermediate that the
-// reference makes between cublasGemmEx and its activation kernel (src/model/ffn.cuh:38-50).
+// up values of 16 features), or relu(x)^2 (a feed-forward without a gate);
+// each saves the round trip of the intermediate that the reference makes between cublasGemmEx and its activation kernel (src/model/ffn.cuh:38-50).
 //
 // Every wait on a barrier is bounded: when a bound is hit the block records an error code, stops
 // taking work, frees its TMEM and returns, so a fault in the hand-over logic cannot hang the GPU.
@@ -44,7 +44,8 @@ constexpr int kThreads = 192;                                   // 6 warps
 constexpr int kTmemCols = 512;
 constexpr int kBandTiles = 16;                                  // 2048 rows of A are shared by the blocks that run together
 
-enum : int { EPI_BF16 = 0, EPI_SILU = 2, EPI_GELU = 3 };      // 2, 3: act(gate) * up with SiLU, with the tanh form of GELU
+// 2, 3: act(gate) * up with SiLU, with the tanh form of GELU; 4: relu(x)^2
+enum : int { EPI_BF16 = 0, EPI_SILU = 2, EPI_GELU = 3, EPI_RELU2 = 4 };
 
 // act(g) * u of the gated epilogues; fast exponential and hyperbolic tangent: the result is rounded to bf16.
 template <int EPI>
@@ -125,7 +126,14 @@ __device__ __forceinline__ void epilogue_tile(bf16* __restrict__ out, uint32_t t
                 uint32_t packed[16];
 #pragma unroll
                 for (int i = 0; i < 32; i += 2) {
-                    const __nv_bfloat162 pk = __floats2bfloat162_rn(__uint_as_float(v[i]), __uint_as_float(v[i + 1]));
+                    float a = __uint_as_float(v[i]), b = __uint_as_float(v[i + 1]);
+                    if (EPI == EPI_RELU2) {
+                        a = fmaxf(a, 0.f);
+                        b = fmaxf(b, 0.f);
+                        a *= a;
+                        b *= b;
+                    }
+                    const __nv_bfloat162 pk = __floats2bfloat162_rn(a, b);
                     packed[i / 2] = *reinterpret_cast<const uint32_t*>(&pk);
                 }
 #pragma unroll
@@ -555,7 +563,9 @@ CPM_API int cpm_gemm_bf16_tcgen05_pair(const void* A, const void* W, void* out, 
         if (N % 32 != 0) return CPM_BAD_ARGUMENT;
         return tc5::launch_pair<tc5::EPI_GELU>(A, W, out, M, N, K, n_blocks, stream);
     }
-    if (epilogue != tc5::EPI_BF16 || N % 8 != 0) return CPM_BAD_ARGUMENT;
+    if (N % 8 != 0) return CPM_BAD_ARGUMENT;
+    if (epilogue == tc5::EPI_RELU2) return tc5::launch_pair<tc5::EPI_RELU2>(A, W, out, M, N, K, n_blocks, stream);
+    if (epilogue != tc5::EPI_BF16) return CPM_BAD_ARGUMENT;
     return tc5::launch_pair<tc5::EPI_BF16>(A, W, out, M, N, K, n_blocks, stream);
 }
 
@@ -576,7 +586,9 @@ CPM_API int cpm_gemm_bf16_tcgen05(const void* A, const void* W, void* out, int M
         if (N % 32 != 0) return CPM_BAD_ARGUMENT;
         return tc5::launch<tc5::EPI_GELU>(A, W, out, M, N, K, n_blocks, stream);
     }
-    if (epilogue != tc5::EPI_BF16 || N % 8 != 0) return CPM_BAD_ARGUMENT;
+    if (N % 8 != 0) return CPM_BAD_ARGUMENT;
+    if (epilogue == tc5::EPI_RELU2) return tc5::launch<tc5::EPI_RELU2>(A, W, out, M, N, K, n_blocks, stream);
+    if (epilogue != tc5::EPI_BF16) return CPM_BAD_ARGUMENT;
     return tc5::launch<tc5::EPI_BF16>(A, W, out, M, N, K, n_blocks, stream);
 }
 

@@ -11,6 +11,8 @@
 //                       the query latent goes on as an activation, the key-value latent into the cache pages, followed
 //                       there by the rotated key part that all heads share (when the design has one)
 //   rotate_heads        turns a range of channels of every head by the token's position
+//   latent_prepare      both of these in one kernel where queries have no latent: the fused projection's rows hold
+//                       [heads x (dim + rot_dim) | rank | rot_dim] (or the queries alone), a token's angles are worked out once
 //   head_project        out[t, h, :] = in[t, h, :] @ w[h]   (w [heads][k][n]; fp32 accumulation), the per-head
 //                       maps Uk^T (queries into the latent space) and Uv (weighted latents into values)
 //   latent_attention    softmax attention of [tokens, heads, rank] fp32 queries over the latent pages (rank up to 1,024); scores,
@@ -23,14 +25,15 @@
 // ---------------------------------------------------------------------------
 // proj rows (fp32, ``stride`` floats) begin [q_rank | rank | rot_dim]: the first two parts are RMS-normed; the third (rot_dim
 // may be 0) is one key part shared by all heads that is turned by the token's position, pairs (c, c + rot_dim/2) or with
-// ``adjacent`` (2c, 2c + 1), angle position * inv_freq[c], and not normed.  The cache row of the token is [rank | rot_dim].
+// ``adjacent`` (2c, 2c + 1), angle position * inv_freq[c], cosine and sine times ``magnitude``, and not normed.  The cache
+// row of the token is [rank | rot_dim].
 template <typename T>
 __global__ void latent_norm_store_kernel(const float* __restrict__ proj, int64_t stride, const float* __restrict__ wq,
                                          const float* __restrict__ wkv, T* __restrict__ cq, T* __restrict__ cache,
                                          const int* __restrict__ positions, const int* __restrict__ token_seq,
                                          const int* __restrict__ slots, const int* __restrict__ page_table, int max_pages,
-                                         int q_rank, int rank, int rot_dim, const float* __restrict__ inv_freq, int adjacent,
-                                         float eps) {
+                                         int q_rank, int rank, int rot_dim, const float* __restrict__ inv_freq, float magnitude,
+                                         int adjacent, float eps) {
     __shared__ float scratch[33];
     pdl_launch_dependents();
     pdl_wait();
@@ -57,6 +60,8 @@ __global__ void latent_norm_store_kernel(const float* __restrict__ proj, int64_t
         const int a = adjacent ? 2 * i : i, b = adjacent ? 2 * i + 1 : i + half;
         float sn = 0.f, cs = 1.f;
         if (inv_freq != nullptr) sincosf((float)p * inv_freq[i], &sn, &cs);
+        sn *= magnitude;
+        cs *= magnitude;
         const float u = row[a], v = row[b];
         dst[a] = from_f32<T>(u * cs - v * sn);
         dst[b] = from_f32<T>(v * cs + u * sn);
@@ -66,27 +71,29 @@ __global__ void latent_norm_store_kernel(const float* __restrict__ proj, int64_t
 CPM_API int cpm_latent_norm_store(const float* proj, int64_t stride, const float* wq, const float* wkv, void* cq, void* cache,
                                   const int* positions, const int* token_seq, const int* slots, const int* page_table,
                                   int max_pages, int n_tokens, int q_rank, int rank, int rot_dim, const float* inv_freq,
-                                  int adjacent, float eps, int dtype, cudaStream_t stream) {
+                                  float magnitude, int adjacent, float eps, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return CPM_OK;
     if (q_rank <= 0 || rank <= 0 || rot_dim < 0 || (rot_dim & 1) || stride < q_rank + rank + rot_dim) return CPM_BAD_ARGUMENT;
     const int threads = (q_rank + rank) >= 1024 ? 256 : 128;
     if (dtype == CPM_BF16)
         cpm_launch(kLaunchRope, latent_norm_store_kernel<bf16>, n_tokens, threads, 0, stream, proj, stride, wq, wkv, (bf16*)cq,
-                   (bf16*)cache, positions, token_seq, slots, page_table, max_pages, q_rank, rank, rot_dim, inv_freq, adjacent, eps);
+                   (bf16*)cache, positions, token_seq, slots, page_table, max_pages, q_rank, rank, rot_dim, inv_freq, magnitude, adjacent,
+                   eps);
     else
         cpm_launch(kLaunchRope, latent_norm_store_kernel<float>, n_tokens, threads, 0, stream, proj, stride, wq, wkv, (float*)cq,
-                   (float*)cache, positions, token_seq, slots, page_table, max_pages, q_rank, rank, rot_dim, inv_freq, adjacent,
+                   (float*)cache, positions, token_seq, slots, page_table, max_pages, q_rank, rank, rot_dim, inv_freq, magnitude, adjacent,
                    eps);
     return launch_status();
 }
 
 // out[t][h][:] = in[t][h][:] (fp32 in, storage type out; heads of ``dh`` channels) with the channels [first, first + rot_dim)
 // of every head turned by the token's position: pairs (c, c + rot_dim/2) or with ``adjacent`` (2c, 2c + 1) counted from
-// ``first``, angle position * inv_freq[c].  One thread per pair or per channel outside the turned part.
+// ``first``, angle position * inv_freq[c], cosine and sine times ``magnitude``.  One thread per pair or per channel outside
+// the turned part.
 template <typename T>
 __global__ void rotate_heads_kernel(const float* __restrict__ in, T* __restrict__ out, const int* __restrict__ positions,
-                                    const float* __restrict__ inv_freq, int64_t n_units, int n_heads, int dh, int first,
-                                    int rot_dim, int adjacent) {
+                                    const float* __restrict__ inv_freq, float magnitude, int64_t n_units, int n_heads, int dh,
+                                    int first, int rot_dim, int adjacent) {
     pdl_launch_dependents();
     pdl_wait();
     const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -105,24 +112,100 @@ __global__ void rotate_heads_kernel(const float* __restrict__ in, T* __restrict_
     const int a = first + (adjacent ? 2 * k : k), b = first + (adjacent ? 2 * k + 1 : k + half);
     float sn, cs;
     sincosf((float)positions[th / n_heads] * inv_freq[k], &sn, &cs);
+    sn *= magnitude;
+    cs *= magnitude;
     const float x = in[base + a], y = in[base + b];
     out[base + a] = from_f32<T>(x * cs - y * sn);
     out[base + b] = from_f32<T>(y * cs + x * sn);
 }
 
-CPM_API int cpm_rotate_heads(const float* in, void* out, const int* positions, const float* inv_freq, int n_tokens, int n_heads,
-                             int dh, int first, int rot_dim, int adjacent, int dtype, cudaStream_t stream) {
+CPM_API int cpm_rotate_heads(const float* in, void* out, const int* positions, const float* inv_freq, float magnitude,
+                             int n_tokens, int n_heads, int dh, int first, int rot_dim, int adjacent, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return CPM_OK;
     if (n_heads < 1 || dh < 1 || first < 0 || rot_dim < 0 || (rot_dim & 1) || first + rot_dim > dh || (rot_dim && !inv_freq))
         return CPM_BAD_ARGUMENT;
     const int64_t n = (int64_t)n_tokens * n_heads * (dh - rot_dim / 2);
     const unsigned blocks = (unsigned)((n + 255) / 256);
     if (dtype == CPM_BF16)
-        cpm_launch(kLaunchRope, rotate_heads_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, in, (bf16*)out, positions, inv_freq, n,
+        cpm_launch(kLaunchRope, rotate_heads_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, in, (bf16*)out, positions, inv_freq, magnitude, n,
                    n_heads, dh, first, rot_dim, adjacent);
     else
         cpm_launch(kLaunchRope, rotate_heads_kernel<float>, dim3(blocks), dim3(256), 0, stream, in, (float*)out, positions, inv_freq,
-                   n, n_heads, dh, first, rot_dim, adjacent);
+                   magnitude, n, n_heads, dh, first, rot_dim, adjacent);
+    return launch_status();
+}
+
+// Queries without a latent: proj rows (fp32, ``stride`` floats) begin [heads x (dim + rot_dim)] and, when ``cache`` is given,
+// go on [rank | rot_dim].  The queries' last rot_dim channels of every head are turned (pairs, angle and magnitude as above)
+// and leave in the storage type; the latent is RMS-normed and stored with the turned key part behind it.  One block a
+// token: its cosines and sines are worked out once and serve all heads and the key part.
+template <typename T>
+__global__ void latent_prepare_kernel(const float* __restrict__ proj, int64_t stride, const float* __restrict__ wkv,
+                                      T* __restrict__ q, T* __restrict__ cache, const int* __restrict__ positions,
+                                      const int* __restrict__ token_seq, const int* __restrict__ slots,
+                                      const int* __restrict__ page_table, int max_pages, int n_heads, int dim, int rank, int rot_dim,
+                                      const float* __restrict__ inv_freq, float magnitude, int adjacent, float eps) {
+    extern __shared__ float lp_smem[];                                   // [half][2] cosine, sine
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, half = rot_dim >> 1, dh = dim + rot_dim;
+    const int p = positions[t];
+    float2* cs = reinterpret_cast<float2*>(lp_smem);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float sn, cn;
+        sincosf((float)p * inv_freq[i], &sn, &cn);
+        cs[i] = make_float2(cn * magnitude, sn * magnitude);
+    }
+    __syncthreads();
+    const float* row = proj + (int64_t)t * stride;
+    T* qrow = q + (int64_t)t * n_heads * dh;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+    const bool vec = ((dim | rot_dim) & 3) == 0 && (stride & 3) == 0;
+    for (int h = warp; h < n_heads; h += n_warps) {
+        const float* src = row + (int64_t)h * dh;
+        T* dst = qrow + (int64_t)h * dh;
+        if (vec) for (int c = 4 * lane; c < dim; c += 128) store4(dst + c, load4(src + c));
+        else for (int c = lane; c < dim; c += 32) dst[c] = from_f32<T>(src[c]);
+        for (int i = lane; i < half; i += 32) {
+            const int a = dim + (adjacent ? 2 * i : i), b = dim + (adjacent ? 2 * i + 1 : i + half);
+            const float u = src[a], v = src[b];
+            dst[a] = from_f32<T>(u * cs[i].x - v * cs[i].y);
+            dst[b] = from_f32<T>(v * cs[i].x + u * cs[i].y);
+        }
+    }
+    if (cache == nullptr) return;
+    row += (int64_t)n_heads * dh;
+    float s = 0.f;
+    for (int c = threadIdx.x; c < rank; c += blockDim.x) s = fmaf(row[c], row[c], s);
+    const float r = 1.0f / sqrtf(block_sum(s, scratch) / (float)rank + eps);
+    const int* pages = page_table + (int64_t)slots[token_seq[t]] * max_pages;
+    const int page = CPM_PAGE(pages, p / kPageTokens, max_pages);
+    T* dst = cache + page_row_offset(page, 0, p % kPageTokens, 1, rank + rot_dim);
+    for (int c = threadIdx.x; c < rank; c += blockDim.x) dst[c] = from_f32<T>(row[c] * r * wkv[c]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const int a = rank + (adjacent ? 2 * i : i), b = rank + (adjacent ? 2 * i + 1 : i + half);
+        const float u = row[a], v = row[b];
+        dst[a] = from_f32<T>(u * cs[i].x - v * cs[i].y);
+        dst[b] = from_f32<T>(v * cs[i].x + u * cs[i].y);
+    }
+}
+
+CPM_API int cpm_latent_prepare(const float* proj, int64_t stride, const float* wkv, void* q, void* cache, const int* positions,
+                               const int* token_seq, const int* slots, const int* page_table, int max_pages, int n_tokens,
+                               int n_heads, int dim, int rank, int rot_dim, const float* inv_freq, float magnitude, int adjacent,
+                               float eps, int dtype, cudaStream_t stream) {
+    if (n_tokens <= 0) return CPM_OK;
+    if (n_heads < 1 || dim < 1 || rank < 1 || rot_dim < 0 || (rot_dim & 1) || rot_dim > 4096 || (rot_dim && !inv_freq)) return CPM_BAD_ARGUMENT;
+    if (stride < (int64_t)n_heads * (dim + rot_dim) + (cache ? rank + rot_dim : 0) || ((uintptr_t)proj & 15)) return CPM_BAD_ARGUMENT;
+    const int threads = (int64_t)n_heads * (dim + rot_dim) >= 1024 ? 256 : 128;
+    const size_t smem = (size_t)rot_dim * sizeof(float) + 16;
+    if (dtype == CPM_BF16)
+        cpm_launch(kLaunchRope, latent_prepare_kernel<bf16>, n_tokens, threads, smem, stream, proj, stride, wkv, (bf16*)q, (bf16*)cache,
+                   positions, token_seq, slots, page_table, max_pages, n_heads, dim, rank, rot_dim, inv_freq, magnitude, adjacent, eps);
+    else
+        cpm_launch(kLaunchRope, latent_prepare_kernel<float>, n_tokens, threads, smem, stream, proj, stride, wkv, (float*)q, (float*)cache,
+                   positions, token_seq, slots, page_table, max_pages, n_heads, dim, rank, rot_dim, inv_freq, magnitude, adjacent, eps);
     return launch_status();
 }
 
@@ -670,19 +753,21 @@ static int launch_latent_mma(const float* q, const void* cache, void* out, int o
     return launch_status();
 }
 
-// bf16 latents, rank a multiple of 16 up to 512; ``out`` fp32, or bf16 with ``out_bf16``; ``scratch``: cpm_latent_attention_scratch_floats floats when n_splits > 1.
+// bf16 latents, rank a multiple of 16 up to 576; ``out`` fp32, or bf16 with ``out_bf16``; ``scratch``: cpm_latent_attention_scratch_floats floats when n_splits > 1.
 CPM_API int cpm_latent_attention_mma(const float* q, const void* cache, void* out, int out_bf16, float* scratch, const int* positions,
                                      const int* token_seq, const int* slots, const int* page_table, int max_pages, int window,
                                      int n_tokens, int n_heads, int rank, float scale, int n_splits, cudaStream_t stream) {
     if (n_tokens <= 0) return CPM_OK;
-    if (n_heads <= 0 || rank <= 0 || rank > 512 || rank % 16 || window < 0 || n_splits < 1 || n_splits > 64) return CPM_BAD_ARGUMENT;
+    if (n_heads <= 0 || rank <= 0 || rank > 576 || rank % 16 || window < 0 || n_splits < 1 || n_splits > 64) return CPM_BAD_ARGUMENT;
     if (n_splits > 1 && scratch == nullptr) return CPM_BAD_ARGUMENT;
     if ((n_heads + kMmaRows - 1) / kMmaRows > 65535) return CPM_BAD_ARGUMENT;
     if (rank <= 128) return launch_latent_mma<4>(q, cache, out, out_bf16, scratch, positions, token_seq, slots, page_table, max_pages, window,
                                                   n_tokens, n_heads, rank, scale, n_splits, stream);
     if (rank <= 256) return launch_latent_mma<8>(q, cache, out, out_bf16, scratch, positions, token_seq, slots, page_table, max_pages, window,
                                                   n_tokens, n_heads, rank, scale, n_splits, stream);
-    return launch_latent_mma<16>(q, cache, out, out_bf16, scratch, positions, token_seq, slots, page_table, max_pages, window, n_tokens,
+    if (rank <= 512) return launch_latent_mma<16>(q, cache, out, out_bf16, scratch, positions, token_seq, slots, page_table, max_pages, window,
+                                                  n_tokens, n_heads, rank, scale, n_splits, stream);
+    return launch_latent_mma<18>(q, cache, out, out_bf16, scratch, positions, token_seq, slots, page_table, max_pages, window, n_tokens,
                                  n_heads, rank, scale, n_splits, stream);
 }
 

@@ -426,7 +426,8 @@ CPM_API int cpm_sigmoid_power(float* z, const float* bias, float tau, int n_toke
 
 // out[t][h][:] = o[t][h][:] / sqrt(mean(o^2) + eps) * weight[:] * act(gate[t][h][:]), act = SiLU or (gate_act 1) the
 // sigmoid, one warp per (token, head);
-// o fp32 [tokens, heads, dv], gate fp32 rows of ``gate_stride`` floats holding [heads, dv], out in the storage type.
+// o fp32 [tokens, heads, dv], gate fp32 rows of ``gate_stride`` floats holding [heads, dv], out in the storage type; weight
+// null: none.
 template <typename T>
 __global__ void gated_head_norm_kernel(const float* __restrict__ o, const float* __restrict__ gate, int64_t gate_stride,
                                        const float* __restrict__ weight, T* __restrict__ out, int heads, int dv, float eps,
@@ -444,7 +445,7 @@ __global__ void gated_head_norm_kernel(const float* __restrict__ o, const float*
     const float f = rsqrtf(warp_sum(ss) / (float)dv + eps);
     const float* gr = gate + t * gate_stride + (int64_t)h * dv;
     for (int c = lane; c < dv; c += 32)
-        out[w * dv + c] = from_f32<T>(row[c] * f * weight[c] * (gate_act == 1 ? sigmoid_acc(gr[c]) : silu_acc(gr[c])));
+        out[w * dv + c] = from_f32<T>(row[c] * f * (weight ? weight[c] : 1.f) * (gate_act == 1 ? sigmoid_acc(gr[c]) : silu_acc(gr[c])));
 }
 
 CPM_API int cpm_gated_head_norm(const float* o, const float* gate, int64_t gate_stride, const float* weight, void* out,

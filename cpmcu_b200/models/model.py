@@ -37,6 +37,8 @@ class Model:
                 written.add(e.lane)
             elif e.lane not in written:
                 raise ValueError(f"a run reads cache lane {e.lane} before any run has written it")
+        # an embedding that keeps something per sequence has a lane behind the layers' lanes
+        self.embedding_lane: Optional[int] = spec.n_lanes() if hasattr(self.embedding, "cache_needs") else None
         self.loaded = False
 
     # ---- weights ----
@@ -91,6 +93,8 @@ class Model:
             if not e.writes_cache and needs[e.lane] is not None and needs[e.lane].kv_heads:
                 # a run that only reads the lane may look further back than the run that writes it
                 needs[e.lane] = needs[e.lane].seen_through(self.blocks[e.layer].cache_needs().window)
+        if self.embedding_lane is not None:
+            needs.append(self.embedding.cache_needs())
         return [n if n is not None else CacheNeeds() for n in needs]
 
     # ---- forward ----
@@ -102,7 +106,11 @@ class Model:
         ops = self.ops
         if not ctx.extras.get("step_begun"):
             ops.begin_step()           # the caller did not lay out the step's workspace itself
-        stream = ResidualStream(ops, self.embedding.forward(ctx.token_ids, ctx.positions))
+        if self.embedding_lane is not None:
+            x, narrow = self.embedding.forward(ctx.token_ids, ctx.positions, ctx, ctx.cache.lane(self.embedding_lane))
+            stream = ResidualStream(ops, x, narrow)
+        else:
+            stream = ResidualStream(ops, self.embedding.forward(ctx.token_ids, ctx.positions))
         if self.spec.streams:
             stream.fan_out(self.spec.streams)      # in the step's persistent part, like the stream itself
         embedded = None

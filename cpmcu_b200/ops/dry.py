@@ -39,6 +39,14 @@ class _NoLibrary:
         return n_tiles * 3 * width
 
     @staticmethod
+    def cpm_retention_tiles_scratch_floats(n_tiles, heads, d, dv):
+        return n_tiles * heads * d * dv
+
+    @staticmethod
+    def cpm_retention_step_sizes(d, dv):
+        return 1
+
+    @staticmethod
     def cpm_listed_attention_tcgen05_max_pages():
         return 11808
 

@@ -57,9 +57,20 @@ _SIGNATURES = {
     "cpm_embed_sinusoid": [_P, _P, _P, _P, _P, c_int, c_int, c_float, c_int, _P],
     "cpm_act_mul": [_P, _P, c_int, c_int, c_int, c_int, c_int, _P],
     "cpm_mingru_scan": [_P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, _P, c_int, c_int, c_int, _P],
-    "cpm_latent_norm_store": [_P, c_int64, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_float,
-                              c_int, _P],
-    "cpm_rotate_heads": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+    "cpm_latent_norm_store": [_P, c_int64, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, c_float, c_int,
+                              c_float, c_int, _P],
+    "cpm_rotate_heads": [_P, _P, _P, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+    "cpm_latent_prepare": [_P, c_int64, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_float, c_int,
+                           c_float, c_int, _P],
+    "cpm_post_norm": [_P, _P, c_float, _P, _P, _P, c_int, c_int, c_float, c_int, _P],
+    "cpm_embed_norm": [_P, _P, c_float, _P, c_int64, c_int64, c_int64, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_float, c_int, _P],
+    "cpm_act_rows": [_P, c_int64, c_int, c_int, _P],
+    "cpm_rotate_scale": [_P, c_int64, _P, c_int, c_int, c_int, c_int, _P, c_float, c_int, c_int, c_float, _P],
+    "cpm_retention_step_sizes": [c_int, c_int],
+    "cpm_retention_step": [_P, c_int64, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, c_float, c_int, c_float, c_float,
+                           c_int, _P],
+    "cpm_retention_tiles": [_P, _P, c_int64, _P, c_int64, _P, c_int64, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, _P, c_int, c_int,
+                            c_int, c_float, c_int, _P],
     "cpm_head_gate": [_P, _P, c_int64, c_int, c_int, c_int, c_int, _P],
     "cpm_channel_decay": [_P, _P, _P, c_int, c_int, c_int, _P],
     "cpm_head_project": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
@@ -170,6 +181,8 @@ def load() -> ctypes.CDLL:
         lib.cpm_decode_attention_scratch_floats.restype = c_int64
         lib.cpm_latent_attention_scratch_floats.argtypes = [c_int, c_int, c_int, c_int]
         lib.cpm_latent_attention_scratch_floats.restype = c_int64
+        lib.cpm_retention_tiles_scratch_floats.argtypes = [c_int, c_int, c_int, c_int]
+        lib.cpm_retention_tiles_scratch_floats.restype = c_int64
         lib.cpm_mingru_summary_floats.argtypes = [c_int, c_int]
         lib.cpm_mingru_summary_floats.restype = c_int64
         for name, argtypes in _SIGNATURES.items():

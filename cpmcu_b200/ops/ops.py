@@ -159,6 +159,57 @@ class Ops:
               f"rmsnorm (hidden {hidden})")
         return y
 
+    def post_norm(self, x: torch.Tensor, a: torch.Tensor, alpha: float, scale: Optional[torch.Tensor], weight: torch.Tensor,
+                  eps: float) -> torch.Tensor:
+        """x <- rms_norm(alpha * x + scale * a) * weight in place (x fp32 [tokens, hidden], a in the compute dtype, scale and
+        weight fp32 [hidden], scale may be None); returns x in the compute dtype (fp32: x itself)."""
+        self._f32(x, "residual stream")
+        self._act(a, "sublayer output")
+        if a.shape != x.shape:
+            raise ValueError(f"sublayer output {tuple(a.shape)} does not match the stream {tuple(x.shape)}")
+        n, hidden = x.shape
+        for t, what in ((scale, "layer scale"), (weight, "norm weight")):
+            if t is not None:
+                self._f32(t, what)
+                if t.numel() != hidden:
+                    raise ValueError(f"{what}: needs [hidden]")
+        y = self.empty(n, hidden) if self.code == BF16 else None
+        check(self.lib.cpm_post_norm(_ptr(x), _ptr(a), float(alpha), _ptr(scale), _ptr(weight), _ptr(y), n, hidden, float(eps),
+                                     self.code, self._stream()), f"post_norm (hidden {hidden})")
+        return x if y is None else y
+
+    def narrowed(self, x: torch.Tensor) -> torch.Tensor:
+        """An fp32 tensor in the compute dtype (fp32: the tensor itself)."""
+        if self.code == F32:
+            return x
+        y = self.empty(*x.shape)
+        y.copy_(x)
+        return y
+
+    def embed_norm(self, ctx, table: torch.Tensor, scale: float, bigram: Optional[torch.Tensor], mul_prev: int, mul_cur: int,
+                   prev_state: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float) -> Tuple[torch.Tensor, torch.Tensor]:
+        """(x fp32 [tokens, hidden], x in the compute dtype) with x = rms_norm(table[id] * scale + bigram[row]) * weight; row =
+        (previous id * mul_prev + id * mul_cur) mod (rows - 1), or the last row for a sequence's first token; the id before
+        a step's first token comes from ``prev_state`` (int32 [slots]), which takes the step's last.  ``bigram`` None: the
+        table alone; ``weight`` None: no norm."""
+        ids = self._i32(ctx.token_ids, "embed ids")
+        self._act(table, "embedding table")
+        n, hidden = ids.numel(), table.shape[1]
+        if bigram is not None:
+            self._act(bigram, "bigram table")
+            self._i32(prev_state, "previous tokens")
+            if bigram.shape[1] != hidden or bigram.shape[0] < 2:
+                raise ValueError("bigram table: needs [buckets + 1, hidden]")
+        if weight is not None:
+            self._f32(weight, "embedding norm weight")
+        x = self.empty(n, hidden, dtype=torch.float32)
+        y = self.empty(n, hidden) if self.code == BF16 else None
+        check(self.lib.cpm_embed_norm(_ptr(ids), _ptr(table), float(scale), _ptr(bigram), bigram.shape[0] - 1 if bigram is not None else 0,
+                                      int(mul_prev), int(mul_cur), _ptr(prev_state), _ptr(ctx.positions), _ptr(ctx.token_seq),
+                                      _ptr(ctx.cu_q), _ptr(ctx.slot_dev), _ptr(weight), _ptr(x), _ptr(y), n, hidden, float(eps),
+                                      self.code, self._stream()), "embed_norm")
+        return x, (x if y is None else y)
+
     def residual_add(self, x: torch.Tensor, delta: torch.Tensor, alpha: float) -> None:
         self._f32(x, "residual stream")
         self._act(delta, "residual addend")
@@ -279,11 +330,11 @@ class Ops:
     # ---- attention over cached latents ----
     def latent_norm_store(self, ctx, proj: torch.Tensor, g_q: torch.Tensor, g_kv: torch.Tensor, lane, q_rank: int,
                           rank: int, eps: float, write_cache: bool = True, rot_dim: int = 0,
-                          inv_freq: Optional[torch.Tensor] = None, adjacent: bool = False) -> torch.Tensor:
+                          inv_freq: Optional[torch.Tensor] = None, adjacent: bool = False, magnitude: float = 1.0) -> torch.Tensor:
         """proj fp32 rows that begin [q_rank | rank | rot_dim]: RMS-norms the first two parts; returns the query latent
         [tokens, q_rank] and stores the key-value latent into the lane's pages at each token's position, followed (with
         ``rot_dim``) by the third part turned by the position: pairs (i, i + rot_dim/2), or (2i, 2i + 1) with ``adjacent``,
-        angle position * inv_freq[i].  A cache row is [rank + rot_dim]."""
+        angle position * inv_freq[i], cosine and sine times ``magnitude``.  A cache row is [rank + rot_dim]."""
         self._f32(proj, "latent projections")
         n = proj.shape[0]
         if proj.shape[1] < q_rank + rank + rot_dim:
@@ -299,21 +350,46 @@ class Ops:
         check(self.lib.cpm_latent_norm_store(_ptr(proj), proj.stride(0), _ptr(g_q), _ptr(g_kv), _ptr(cq), _ptr(cache),
                                              _ptr(ctx.positions), _ptr(ctx.token_seq), _ptr(ctx.slot_dev), _ptr(lane.page_table),
                                              lane.page_table.shape[1], n, q_rank, rank, int(rot_dim),
-                                             _ptr(inv_freq) if rot_dim else None, 1 if adjacent else 0, float(eps), self.code,
-                                             self._stream()), "latent_norm_store")
+                                             _ptr(inv_freq) if rot_dim else None, float(magnitude), 1 if adjacent else 0, float(eps),
+                                             self.code, self._stream()), "latent_norm_store")
         return cq
 
     def rotate_heads(self, ctx, x: torch.Tensor, n_heads: int, first: int, rot_dim: int, inv_freq: torch.Tensor,
-                     adjacent: bool = False) -> torch.Tensor:
+                     adjacent: bool = False, magnitude: float = 1.0) -> torch.Tensor:
         """x fp32 [tokens, heads * dh] -> [tokens, heads * dh] in the compute dtype with the channels [first, first +
         rot_dim) of every head turned by the token's position (pairs as in ``latent_norm_store``)."""
         self._f32(x, "heads to rotate")
         self._f32(inv_freq, "inv_freq")
         n, dh = x.shape[0], x.shape[1] // n_heads
         out = self.empty(n, n_heads * dh)
-        check(self.lib.cpm_rotate_heads(_ptr(x), _ptr(out), _ptr(ctx.positions), _ptr(inv_freq), n, n_heads, dh, int(first),
-                                        int(rot_dim), 1 if adjacent else 0, self.code, self._stream()), "rotate_heads")
+        check(self.lib.cpm_rotate_heads(_ptr(x), _ptr(out), _ptr(ctx.positions), _ptr(inv_freq), float(magnitude), n, n_heads, dh,
+                                        int(first), int(rot_dim), 1 if adjacent else 0, self.code, self._stream()), "rotate_heads")
         return out
+
+    def latent_prepare(self, ctx, proj: torch.Tensor, g_kv: Optional[torch.Tensor], lane, n_heads: int, dim: int, rank: int,
+                       rot_dim: int, inv_freq: Optional[torch.Tensor], eps: float, write_cache: bool = True,
+                       adjacent: bool = False, magnitude: float = 1.0) -> torch.Tensor:
+        """proj fp32 rows that begin [heads * (dim + rot_dim)] and, with ``write_cache``, go on [rank | rot_dim] (queries
+        without a latent of their own): returns the queries [tokens, heads * (dim + rot_dim)] in the compute dtype, the last
+        rot_dim channels of every head turned as in ``latent_norm_store``, and with ``write_cache`` norms the latent and
+        stores it and the turned key part into the lane's pages."""
+        self._f32(proj, "latent projections")
+        n, cols = proj.shape[0], n_heads * (dim + rot_dim)
+        if proj.shape[1] < cols + (rank + rot_dim if write_cache else 0):
+            raise ValueError("latent_prepare: the projections' row size does not match the head counts")
+        if rot_dim:
+            self._f32(inv_freq, "inv_freq")
+            if inv_freq.numel() != rot_dim // 2:
+                raise ValueError("inv_freq needs rot_dim/2 entries")
+        if write_cache and lane.k.shape[-1] != rank + rot_dim:
+            raise ValueError(f"latent_prepare: the lane's rows hold {lane.k.shape[-1]} values, not {rank + rot_dim}")
+        q = self.empty(n, cols)
+        check(self.lib.cpm_latent_prepare(_ptr(proj), proj.stride(0), _ptr(g_kv), _ptr(q), _ptr(lane.k) if write_cache else None,
+                                          _ptr(ctx.positions), _ptr(ctx.token_seq), _ptr(ctx.slot_dev), _ptr(lane.page_table),
+                                          lane.page_table.shape[1], n, n_heads, dim, rank, int(rot_dim),
+                                          _ptr(inv_freq) if rot_dim else None, float(magnitude), 1 if adjacent else 0, float(eps),
+                                          self.code, self._stream()), "latent_prepare")
+        return q
 
     def head_gate(self, x: torch.Tensor, gate: torch.Tensor, n_heads: int) -> torch.Tensor:
         """In place: x [tokens, heads * dv] (compute dtype) times sigmoid(gate [tokens, heads]) head by head; the gate is
@@ -367,7 +443,7 @@ class Ops:
         return max(1, min(self.LATENT_MAX_SPLITS, 3 * self.sm_count // blocks, ((keys + 31) // 32) // 2))
 
     def latent_attention_on_tensor_cores(self, rank: int) -> bool:
-        return self.code == BF16 and rank % 16 == 0 and rank <= 512
+        return self.code == BF16 and rank % 16 == 0 and rank <= 576
 
     def latent_attention(self, ctx, q_lat: torch.Tensor, lane, scale: float, window: int = 0,
                          n_splits: Optional[int] = None, tensor_cores: Optional[bool] = None,
@@ -382,7 +458,7 @@ class Ops:
         narrow = bool(out_compute_dtype) and mma_ok and tensor_cores is not False
         out = self.empty(n, H, R, dtype=self.dtype if narrow else torch.float32)
         if tensor_cores and not mma_ok:
-            raise ValueError("the tensor-core latent attention takes bf16 latents of a rank that is a multiple of 16 up to 512")
+            raise ValueError("the tensor-core latent attention takes bf16 latents of a rank that is a multiple of 16 up to 576")
         if mma_ok and tensor_cores is not False:
             if n_splits is None:
                 n_splits = self.latent_attention_splits(ctx, n, H, int(window))
@@ -461,10 +537,10 @@ class Ops:
             torch.mm(a, w.t(), out_dtype=c.dtype, out=c)
 
     def linear_tcgen05(self, a: torch.Tensor, w: torch.Tensor, gated: bool = False, pair: bool = False,
-                       epilogue: int = 2) -> torch.Tensor:
+                       epilogue: Optional[int] = None) -> torch.Tensor:
         """a[M,K] @ w[N,K]^T on the tcgen05 tensor cores (TMA operands, TMEM accumulator); with ``gated`` the
         weight is a gate_up matrix interleaved in blocks of 8 and the result is act(gate) * up, [M, N/2] (``epilogue`` 2:
-        SiLU, 3: the tanh form of GELU).
+        SiLU, the default, 3: the tanh form of GELU); without, ``epilogue`` 4 gives relu(x)^2.
         ``pair``: two blocks work on one 256 x 256 tile (cta_group::2)."""
         self._act(a, "linear input")
         self._act(w, "linear weight")
@@ -472,7 +548,7 @@ class Ops:
         N = w.shape[0]
         out = self.empty(M, N // 2 if gated else N)
         entry = self.lib.cpm_gemm_bf16_tcgen05_pair if pair else self.lib.cpm_gemm_bf16_tcgen05
-        check(entry(_ptr(a), _ptr(w), _ptr(out), M, N, K, int(epilogue) if gated else 0, self.sm_count, self._stream()),
+        check(entry(_ptr(a), _ptr(w), _ptr(out), M, N, K, int(epilogue if epilogue is not None else (2 if gated else 0)), self.sm_count, self._stream()),
               f"tcgen05 matrix product [{M}x{K}] x [{N}x{K}]^T")
         return out
 
@@ -512,6 +588,28 @@ class Ops:
         if activation == 0:
             return self.silu_mul(self.linear(a, w_gate_up), interleave)
         return self.act_mul(self.linear(a, w_gate_up), interleave, activation)
+
+    RELU2, RELU2_EPILOGUE = 2, 4      # the activation kernels' code of relu(x)^2 and the product kernels' epilogue
+
+    def relu2_linear(self, a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        """relu(a @ w^T)^2 for w [N, K].  The weight-streaming product (few rows) and the tcgen05 product (many rows) apply it
+        in their epilogues; otherwise a kernel of its own follows the product."""
+        M, K = a.shape
+        N = w.shape[0]
+        if self._skinny_ok(M, K, N):
+            self._act(a, "linear input")
+            self._act(w, "linear weight")
+            h = self.empty(M, N)
+            check(self.lib.cpm_gemm_skinny_bf16(_ptr(w), _ptr(a), _ptr(h), M, N, K, 1.0, self.RELU2_EPILOGUE, self._stream()),
+                  "skinny matrix product with relu^2")
+            return h
+        few_tiles = M < 256 and N // 256 < self.sm_count // 2
+        if (self.code == BF16 and self.use_tcgen05 and M >= self.TCGEN05_MIN_ROWS and K % 64 == 0 and N % 8 == 0
+                and a.data_ptr() % 16 == 0 and not few_tiles):
+            return self.linear_tcgen05(a, w, pair=self.tcgen05_pair, epilogue=self.RELU2_EPILOGUE)
+        h = self.linear(a, w)
+        check(self.lib.cpm_act_rows(_ptr(h), h.numel(), self.RELU2, self.code, self._stream()), "relu^2")
+        return h
 
     # ---- attention ----
     def rope_store(self, qkv: torch.Tensor, n_heads: int, n_kv: int, d: int, positions: torch.Tensor,
@@ -899,18 +997,95 @@ class Ops:
         check(self.lib.cpm_sigmoid_power(_ptr(z), _ptr(bias), float(tau), z.shape[0], z.shape[1], self._stream()), "sigmoid_power")
         return z
 
-    def gated_head_norm(self, o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float,
+    def gated_head_norm(self, o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], eps: float,
                         gate_activation: str = "silu") -> torch.Tensor:
-        """o fp32 [tokens, heads, dv], gate fp32 [tokens, heads*dv] (may be a slice of wider rows), weight fp32 [dv] ->
+        """o fp32 [tokens, heads, dv], gate fp32 [tokens, heads*dv] (may be a slice of wider rows), weight fp32 [dv] or None ->
         rms_norm(o) * weight * act(gate) per head (act: "silu" or "sigmoid"), [tokens, heads*dv] in the compute dtype."""
         self._f32(o, "recurrence output")
-        self._f32(weight, "head norm weight")
+        if weight is not None:
+            self._f32(weight, "head norm weight")
         n, heads, dv = o.shape
         if gate.dtype != torch.float32 or gate.shape != (n, heads * dv) or gate.stride(1) != 1:
             raise ValueError("gated_head_norm: the gate must be fp32 [tokens, heads*dv]")
         out = self.empty(n, heads * dv)
         check(self.lib.cpm_gated_head_norm(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(out), n, heads, dv, float(eps),
                                            {"silu": 0, "sigmoid": 1}[gate_activation], self.code, self._stream()), "gated_head_norm")
+        return out
+
+    # ---- linear attention with one fixed decay per head ----
+    RETENTION_TILE_MIN_TOKENS = 16      # portions shorter than this walk token by token (a tile of 64 would be mostly empty)
+
+    def rotate_scale(self, ctx, x: torch.Tensor, heads: int, d: int, inv_freq: Optional[torch.Tensor], rot_dim: int,
+                     magnitude: float = 1.0, adjacent: bool = False, first_scaled: Optional[int] = None, factor: float = 1.0) -> None:
+        """In place on fp32 rows (unit stride inside a row) that begin with ``heads`` heads of ``d`` channels: the first
+        ``rot_dim`` channels of each are turned by the token's position (pairs (i, i + rot_dim/2), or (2i, 2i + 1) with
+        ``adjacent``; cosine and sine times ``magnitude``), and the heads from ``first_scaled`` on are multiplied by ``factor``."""
+        if x.dtype != torch.float32 or x.dim() != 2 or x.stride(1) != 1 or x.shape[1] < heads * d:
+            raise ValueError("rotate_scale: needs fp32 rows with unit stride inside a row")
+        if rot_dim:
+            self._f32(inv_freq, "inv_freq")
+            if inv_freq.numel() != rot_dim // 2:
+                raise ValueError("inv_freq needs rot_dim/2 entries")
+        check(self.lib.cpm_rotate_scale(_ptr(x), x.stride(0), _ptr(ctx.positions), x.shape[0], heads, d, int(rot_dim),
+                                        _ptr(inv_freq) if rot_dim else None, float(magnitude), 1 if adjacent else 0,
+                                        heads if first_scaled is None else int(first_scaled), float(factor), self._stream()),
+              "rotate_scale")
+
+    def retention_step(self, ctx, proj: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, heads: int, d: int, dv: int,
+                       inv_freq: Optional[torch.Tensor], rot_dim: int, magnitude: float, adjacent: bool, k_factor: float,
+                       eps: float) -> torch.Tensor:
+        """A decode step of the whole mixer between its products, in one kernel: proj fp32 [tokens, 2 heads (d + dv)] =
+        [q | k | v | gate], one token per sequence; q and k are turned, k scaled, the state [slots, heads, d, dv] decayed
+        (decay fp32 [heads]), added to and read, each head's read-out normed and multiplied by SiLU of the gate ->
+        [tokens, heads * dv] in the compute dtype."""
+        self._f32(proj, "retention projections")
+        self._f32(decay, "decay")
+        self._f32(state, "retention state")
+        n = proj.shape[0]
+        if proj.shape[1] != 2 * heads * (d + dv) or decay.numel() != heads or tuple(state.shape[1:]) != (heads, d, dv):
+            raise ValueError("retention_step: projections [tokens, 2 heads (d + dv)], decay [heads], state [slots, heads, d, dv]")
+        out = self.empty(n, heads * dv)
+        check(self.lib.cpm_retention_step(_ptr(proj), proj.stride(0), _ptr(decay), _ptr(state), _ptr(ctx.positions), _ptr(ctx.token_seq),
+                                          _ptr(ctx.slot_dev), _ptr(out), n, heads, d, dv, int(rot_dim),
+                                          _ptr(inv_freq) if rot_dim else None, float(magnitude), 1 if adjacent else 0,
+                                          float(k_factor), float(eps), self.code, self._stream()),
+              f"retention_step ({heads} heads, {d} x {dv})")
+        return out
+
+    def retention_step_ok(self, ctx, d: int, dv: int) -> bool:
+        return bool(ctx.is_decode) and bool(self.lib.cpm_retention_step_sizes(d, dv))
+
+    def retention_tiles_ok(self, ctx, d: int, dv: int) -> bool:
+        return (not ctx.is_decode and ctx.q_tiles is not None and ctx.max_q_len >= self.RETENTION_TILE_MIN_TOKENS
+                and d <= 256 and dv <= 256)
+
+    def retention_tiles(self, ctx, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: Optional[torch.Tensor],
+                        powers: torch.Tensor, state: torch.Tensor, heads: int, d: int, dv: int, eps: float = 0.0) -> torch.Tensor:
+        """The recurrence S <- a_h S + k v^T, o = S^T q over a prompt's tiles of 64 tokens (``ctx.q_tiles``), in 32-bit:
+        q, k fp32 views [tokens, heads * d], v [tokens, heads * dv] (slices of wider rows), powers fp32 [heads, 65] = a_h^0 ..
+        a_h^64, state fp32 [slots, heads, d, dv], read at a sequence's first token of the step (zeros at position 0) and
+        written at its last.  With ``gate`` (fp32 [tokens, heads * dv], a slice of wider rows): o / rms(o) * silu(gate) per
+        head, [tokens, heads * dv] in the compute dtype; without: o, fp32 [tokens, heads, dv]."""
+        n = q.shape[0]
+        for t, what, width in ((q, "q", heads * d), (k, "k", heads * d), (v, "v", heads * dv)) + \
+                (((gate, "gate", heads * dv),) if gate is not None else ()):
+            if t.dtype != torch.float32 or t.shape != (n, width) or t.stride(1) != 1:
+                raise ValueError(f"retention_tiles: {what} must be fp32 [tokens, {width}] with unit stride inside a row")
+        if q.stride(0) != k.stride(0):
+            raise ValueError("retention_tiles: q and k must have the same row stride")
+        self._f32(powers, "decay powers")
+        self._f32(state, "retention state")
+        if tuple(powers.shape) != (heads, QUERY_TILE_TOKENS + 1) or tuple(state.shape[1:]) != (heads, d, dv):
+            raise ValueError(f"retention_tiles: powers [heads, {QUERY_TILE_TOKENS + 1}], state [slots, heads, d, dv]")
+        tile_seq, tile_row, n_tiles = ctx.q_tiles
+        out = self.empty(n, heads * dv) if gate is not None else self.empty(n, heads, dv, dtype=torch.float32)
+        scratch = self.empty(int(self.lib.cpm_retention_tiles_scratch_floats(n_tiles, heads, d, dv)), dtype=torch.float32)
+        check(self.lib.cpm_retention_tiles(_ptr(q), _ptr(k), q.stride(0), _ptr(v), v.stride(0), _ptr(gate),
+                                           gate.stride(0) if gate is not None else 0, _ptr(powers), _ptr(state), _ptr(ctx.positions),
+                                           _ptr(ctx.cu_q), _ptr(ctx.slot_dev), _ptr(tile_seq), _ptr(tile_row), int(n_tiles), ctx.n_seqs,
+                                           _ptr(scratch), _ptr(out), heads, d, dv, float(eps), self.code, self._stream()),
+              f"retention_tiles ({heads} heads, {d} x {dv})")
+        LAUNCHES_EXTRA[0] += 2
         return out
 
     GATE_ACTIVATIONS = {"silu": 0, "sigmoid": 1}

@@ -278,9 +278,11 @@ class ResidualStream:
     src/model/norm.cuh:53-99); the sum itself is always kept and formed in 32-bit.
     """
 
-    def __init__(self, ops, x: torch.Tensor):
+    def __init__(self, ops, x: torch.Tensor, narrow: Optional[torch.Tensor] = None):
         self.ops = ops
         self.x = x
+        # x in the compute dtype, where the kernel that wrote x last left that too (None: nobody did)
+        self.narrow: Optional[torch.Tensor] = narrow
         self.pending: Optional[torch.Tensor] = None
         self.pending2: Optional[torch.Tensor] = None       # a second output with the same factor (two sublayers side by side)
         self.pending_scale: float = 1.0
@@ -297,6 +299,7 @@ class ResidualStream:
     def add(self, delta: torch.Tensor, scale: float = 1.0, second: Optional[torch.Tensor] = None) -> None:
         """x += scale * delta (+ scale * second), deferred to the next norm's pass or the next ``flush``."""
         self.flush()
+        self.narrow = None
         self.pending = delta
         self.pending2 = second
         self.pending_scale = float(scale)
@@ -313,6 +316,13 @@ class ResidualStream:
                 self.ops.residual_add(self.x, self.pending2, self.pending_scale)
             self.pending = self.pending2 = None
         return self.x
+
+    def itself(self) -> torch.Tensor:
+        """The stream in the compute dtype, for a sublayer that reads it without a norm in front."""
+        x = self.flush()
+        if self.narrow is None or self.copies is not None:
+            self.narrow = self.ops.narrowed(x)
+        return self.narrow
 
     def normed(self, norm: Norm, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         if self.copies is not None:

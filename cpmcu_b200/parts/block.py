@@ -56,6 +56,61 @@ class ParallelResidualBlock(Block):
         stream.add(a, self.residual_scale, second=f)
 
 
+@BLOCKS.register("post_norm_residual")
+class PostNormResidualBlock(Block):
+    """The norm after the sum: x <- norm1(alpha * x + s1 * mixer(x)); x <- norm2(alpha * x + s2 * feed_forward(x)).
+
+    A sublayer reads the stream itself (in the compute dtype), and what the layer leaves is normed.  alpha is one constant
+    (``alpha``); s1 and s2 are one number per channel (``layer_scale``; tensors ``names["mixer_scale"]`` and
+    ``names["feed_forward_scale"]`` [hidden]), or absent.  One kernel a sublayer scales, adds, norms, keeps the 32-bit
+    stream and leaves the copy in the compute dtype that the next sublayer's products read.  A layer without a
+    feed-forward has the first half only.
+    """
+
+    recordable_prompt = True
+
+    def __init__(self, ops, mixer, feed_forward, mixer_norm, feed_forward_norm, names, hidden_size: int, alpha: float = 1.0,
+                 layer_scale: bool = True):
+        super().__init__(ops, mixer, feed_forward, mixer_norm, feed_forward_norm, names)
+        if feed_forward is not None and feed_forward_norm is None:
+            raise ValueError("post_norm_residual: a feed-forward needs its norm")
+        for n in (mixer_norm, feed_forward_norm):
+            if n is not None and not hasattr(n, "post_forward"):
+                raise ValueError("post_norm_residual needs norms that offer post_forward (rms_norm)")
+        self.hidden_size, self.alpha, self.layer_scale = int(hidden_size), float(alpha), bool(layer_scale)
+        self.scales = [None, None]
+
+    def _scale_names(self):
+        if not self.layer_scale:
+            return []
+        names = [self.names.get("mixer_scale", "mixer_scale")]
+        if self.feed_forward is not None:
+            names.append(self.names.get("feed_forward_scale", "feed_forward_scale"))
+        return names
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        out = super().weight_specs()
+        for name in self._scale_names():
+            out[name] = WeightSpec((self.hidden_size,), "vector")
+        return out
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        super().load_weights(tensors)
+        for i, name in enumerate(self._scale_names()):
+            self.scales[i] = self.ops.keep(tensors[name].float().contiguous())
+
+    def weight_bytes(self) -> int:
+        return super().weight_bytes() + 4 * self.hidden_size * len(self._scale_names())
+
+    def forward(self, ctx, stream: ResidualStream, lane, writes_cache: bool) -> None:
+        a = self.mixer.forward(ctx, stream.itself(), lane, writes_cache)
+        stream.narrow = self.mixer_norm.post_forward(stream.x, a, self.alpha, self.scales[0])
+        if self.feed_forward is None:
+            return
+        f = self.feed_forward.forward(ctx, stream.narrow)
+        stream.narrow = self.feed_forward_norm.post_forward(stream.x, f, self.alpha, self.scales[1])
+
+
 @BLOCKS.register("sandwich_norm_shift")
 class SandwichNormShiftBlock(Block):
     """x += post1(mixer(shift(pre1(x)))); x += post2(feed_forward(pre2(x))): a norm before and after each sublayer,

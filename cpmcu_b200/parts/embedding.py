@@ -11,7 +11,7 @@ from typing import Dict, Optional, Type
 
 import torch
 
-from .base import Part, Registry, WeightSpec
+from .base import CacheNeeds, Part, Registry, WeightSpec
 
 EMBEDDINGS: Registry[Type[Part]] = Registry("embedding")
 HEADS: Registry[Type[Part]] = Registry("output head")
@@ -68,6 +68,54 @@ class SinusoidalScaledEmbedding(Part):
         if positions is None:
             raise ValueError("sinusoidal_scaled_embedding needs the tokens' positions")
         return self.ops.embed_sinusoid(token_ids, positions, self.weight, self.freq, self.scale)
+
+
+@EMBEDDINGS.register("bigram_embedding")
+class BigramEmbedding(Part):
+    """norm(table[id] * scale + bigram[row]): besides its own row a token takes a row of a second table that a hash of the
+    token before it and of the token itself picks,
+
+        row = (previous id * mul_prev + id * mul_cur) mod buckets,    or row ``buckets`` (the last) for a first token,
+
+    and the sum passes through an RMS norm with weight.  ``buckets`` 0: no second table; ``norm_name`` None: no norm.  The
+    previous id is per-sequence state (``previous_token``, int32), so a sequence goes on the same way however its tokens
+    are cut into steps.  Tables, hash, sum and norm are one kernel, which leaves the stream in 32-bit and in the compute dtype.
+    An embedding with state has a cache lane of its own (``cache_needs``) and is called with the step's context."""
+
+    recordable_prompt = True
+
+    def __init__(self, ops, vocab_size: int, hidden_size: int, scale: float = 1.0, buckets: int = 0, mul_prev: int = 1, mul_cur: int = 1,
+                 eps: float = 1e-5, weight_name: str = "weight", bigram_name: str = "bigram", norm_name: Optional[str] = "norm"):
+        super().__init__(ops)
+        self.vocab_size, self.hidden_size, self.scale = int(vocab_size), int(hidden_size), float(scale)
+        self.buckets, self.mul_prev, self.mul_cur, self.eps = int(buckets or 0), int(mul_prev), int(mul_cur), float(eps)
+        self.weight_name, self.bigram_name, self.norm_name = str(weight_name), str(bigram_name), norm_name
+        self.weight: Optional[torch.Tensor] = None
+        self.bigram: Optional[torch.Tensor] = None
+        self.norm: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        out = {self.weight_name: WeightSpec((self.vocab_size, self.hidden_size))}
+        if self.buckets:
+            out[self.bigram_name] = WeightSpec((self.buckets + 1, self.hidden_size))
+        if self.norm_name is not None:
+            out[self.norm_name] = WeightSpec((self.hidden_size,), "vector")
+        return out
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight = self.ops.keep(tensors[self.weight_name].contiguous())
+        if self.buckets:
+            self.bigram = self.ops.keep(tensors[self.bigram_name].contiguous())
+        if self.norm_name is not None:
+            self.norm = self.ops.keep(tensors[self.norm_name].float().contiguous())
+
+    def cache_needs(self) -> CacheNeeds:
+        return CacheNeeds(state={"previous_token": ((), torch.int32)} if self.buckets else {})
+
+    def forward(self, token_ids: torch.Tensor, positions: Optional[torch.Tensor] = None, ctx=None, lane=None):
+        """Returns (stream fp32, the same in the compute dtype)."""
+        state = lane.state["previous_token"] if self.buckets else None
+        return self.ops.embed_norm(ctx, self.weight, self.scale, self.bigram, self.mul_prev, self.mul_cur, state, self.norm, self.eps)
 
 
 @HEADS.register("scaled_lm_head")

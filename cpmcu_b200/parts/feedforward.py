@@ -66,6 +66,37 @@ class GatedFeedForward(FeedForward):
         return self.ops.linear(h, self.w_down)
 
 
+@FEED_FORWARDS.register("plain_ffn")
+class PlainFeedForward(FeedForward):
+    """A feed-forward without a gate: down( relu(up y)^2 ).  ``names``: the matrices' names below the part's prefix, by "up"
+    and "down".  The activation (32-bit, on the product's accumulator) is applied in the product's epilogue."""
+
+    recordable_prompt = True
+
+    def __init__(self, ops, hidden_size: int, intermediate_size: int, activation: str = "relu2", names=None):
+        super().__init__(ops)
+        if activation != "relu2":
+            raise ValueError(f"plain_ffn: activation '{activation}' is not built; known: ['relu2']")
+        self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        self.names = dict({"up": "up_proj.weight", "down": "down_proj.weight"}, **(dict(names) if names else {}))
+        self.w_up: Optional[torch.Tensor] = None
+        self.w_down: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        i, h = self.intermediate_size, self.hidden_size
+        return {self.names["up"]: WeightSpec((i, h)), self.names["down"]: WeightSpec((h, i))}
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.w_up = self.ops.keep(tensors[self.names["up"]].contiguous())
+        self.w_down = self.ops.keep(tensors[self.names["down"]].contiguous())
+
+    def weight_bytes(self) -> int:
+        return (self.w_up.numel() + self.w_down.numel()) * self.w_up.element_size()
+
+    def forward(self, ctx, y: torch.Tensor) -> torch.Tensor:
+        return self.ops.linear(self.ops.relu2_linear(y, self.w_up), self.w_down)
+
+
 @FEED_FORWARDS.register("routed_experts")
 class RoutedExperts(FeedForward):
     """A mixture of gated feed-forward experts, of which every token uses ``top``:

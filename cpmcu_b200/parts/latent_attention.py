@@ -28,17 +28,23 @@ class LatentAttention(Mixer):
     channels) and the score is (q_plain . k_plain + q_turned . k_turned) * scale.  The cached row of a token is then
     [c | turned key part], the query in latent space [Wuk_h^T q_plain | q_turned], and the turned part's columns of the
     weighted sum of rows are dropped by the value map (zero rows in its matrix): still one row per token, nothing
-    decompressed.  With ``gate`` head h's output is multiplied by sigmoid(Wg h)_h before Wo.
+    decompressed.  With ``gate`` head h's output is multiplied by sigmoid(Wg h)_h before Wo.  A position encoding with a
+    magnitude factor has it on cosine and sine, of the queries and of the key part alike.
+
+    ``q_rank`` 0: queries have no latent, q = Wq h (tensor ``names["q"]``); one product gives the queries and the latent's
+    row, and one kernel turns the queries, norms the latent and stores it.  ``own_kv`` False: the layer has no Wdkv and
+    reads the rows (latent and turned key part) that another layer of equal ``kv_rank``, ``rot_dim`` and rotation cached,
+    through its own queries, Wuk, Wuv and scale.
     """
 
     recordable_prompt = True
 
     DEFAULT_NAMES = {"dq": "dq.weight", "dq_norm": "dq_norm.weight", "uq": "uq.weight", "dkv": "dkv.weight",
-                     "dkv_norm": "dkv_norm.weight", "uk": "uk.weight", "uv": "uv.weight", "o": "o.weight", "gate": "g"}
+                     "dkv_norm": "dkv_norm.weight", "uk": "uk.weight", "uv": "uv.weight", "o": "o.weight", "gate": "g", "q": "q.weight"}
 
     def __init__(self, ops, hidden_size: int, n_heads: int, head_dim: int, value_dim: int, q_rank: int, kv_rank: int,
                  softmax_scale: float, eps: float, window: Optional[int] = None, names=None, rot_dim: int = 0,
-                 position: Optional[PartSpec] = None, gate: bool = False):
+                 position: Optional[PartSpec] = None, gate: bool = False, own_kv: bool = True):
         super().__init__(ops)
         self.hidden_size, self.n_heads, self.d, self.vd = int(hidden_size), int(n_heads), int(head_dim), int(value_dim)
         self.q_rank, self.kv_rank = int(q_rank), int(kv_rank)
@@ -48,20 +54,31 @@ class LatentAttention(Mixer):
         self.row = self.kv_rank + self.rot_dim                    # what the cache keeps of a token
         if self.row > 1024:
             raise ValueError(f"latent_attention: a cached row of {self.row} values is beyond the 1,024 the attention kernels keep per head")
-        self.inv_freq, self.adjacent = None, False
+        self.own_kv = bool(own_kv)
+        if not self.own_kv and (self.q_rank or self.gate):
+            raise ValueError("latent_attention: a layer that reads another's rows is built for queries without a latent and no gate")
+        if not self.q_rank and self.gate:
+            raise ValueError("latent_attention: the gate is built for queries with a latent")
+        self.inv_freq, self.adjacent, self.magnitude = None, False, 1.0
         if self.rot_dim:
             if position is None:
                 raise ValueError("latent_attention: a rotated part needs a position encoding")
             enc = build_part(POSITIONS, position, ops)
             rot = enc.rotary()
-            if rot is None or rot[1] != 1.0 or rot[2] != self.rot_dim:
+            if rot is None or rot[2] != self.rot_dim:
                 raise ValueError("latent_attention: the position encoding must be a rotation of pairs over all rot_dim channels")
-            self.inv_freq, self.adjacent = rot[0], bool(getattr(enc, "adjacent", False))
+            self.inv_freq, self.magnitude, self.adjacent = rot[0], float(rot[1]), bool(getattr(enc, "adjacent", False))
         self.names = dict(self.DEFAULT_NAMES, **(dict(names) if names else {}))
         self.w_down = self.w_uq = self.w_uk = self.w_uv = self.w_o = self.g_q = self.g_kv = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         n, H, h = self.names, self.n_heads, self.hidden_size
+        if not self.q_rank:
+            out = {n["q"]: WeightSpec((H * (self.d + self.rot_dim), h)), n["uk"]: WeightSpec((H * self.d, self.kv_rank)),
+                   n["uv"]: WeightSpec((H * self.vd, self.kv_rank)), n["o"]: WeightSpec((h, H * self.vd))}
+            if self.own_kv:
+                out.update({n["dkv"]: WeightSpec((self.row, h)), n["dkv_norm"]: WeightSpec((self.kv_rank,), "vector")})
+            return out
         out = {n["dq"]: WeightSpec((self.q_rank, h)), n["dq_norm"]: WeightSpec((self.q_rank,), "vector"),
                n["uq"]: WeightSpec((H * (self.d + self.rot_dim), self.q_rank)), n["dkv"]: WeightSpec((self.row, h)),
                n["dkv_norm"]: WeightSpec((self.kv_rank,), "vector"), n["uk"]: WeightSpec((H * self.d, self.kv_rank)),
@@ -72,9 +89,12 @@ class LatentAttention(Mixer):
 
     def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
         n, H, keep = self.names, self.n_heads, self.ops.keep
-        down = [tensors[n["dq"]], tensors[n["dkv"]]] + ([tensors[n["gate"]]] if self.gate else [])
-        self.w_down = keep(torch.cat(down, dim=0).contiguous())      # one product for both latents (and the gates' logits)
-        self.w_uq = keep(tensors[n["uq"]].contiguous())
+        if self.q_rank:
+            down = [tensors[n["dq"]], tensors[n["dkv"]]] + ([tensors[n["gate"]]] if self.gate else [])
+            self.w_uq = keep(tensors[n["uq"]].contiguous())
+        else:
+            down = [tensors[n["q"]]] + ([tensors[n["dkv"]]] if self.own_kv else [])
+        self.w_down = keep(torch.cat(down, dim=0).contiguous())      # one product of the layer's input for all that reads it
         # per head [k][n] matrices for in[t, h, :] @ w[h]: Wuk_h is [dim, rank] as stored; Wuv_h [vdim, rank] is transposed
         uk = tensors[n["uk"]].view(H, self.d, self.kv_rank)
         uv = tensors[n["uv"]].view(H, self.vd, self.kv_rank).transpose(1, 2)
@@ -91,12 +111,15 @@ class LatentAttention(Mixer):
         self.w_uk = keep(uk.contiguous())
         self.w_uv = keep(uv.contiguous())
         self.w_o = keep(tensors[n["o"]].contiguous())
-        self.g_q = keep(tensors[n["dq_norm"]].float().contiguous())
-        self.g_kv = keep(tensors[n["dkv_norm"]].float().contiguous())
+        if self.q_rank:
+            self.g_q = keep(tensors[n["dq_norm"]].float().contiguous())
+        if self.own_kv:
+            self.g_kv = keep(tensors[n["dkv_norm"]].float().contiguous())
 
     def weight_bytes(self) -> int:
         mats = (self.w_down, self.w_uq, self.w_uk, self.w_uv, self.w_o)
-        return sum(m.numel() for m in mats) * self.w_o.element_size() + 4 * (self.q_rank + self.kv_rank)
+        return sum(m.numel() for m in mats if m is not None) * self.w_o.element_size() + \
+            4 * (self.q_rank + (self.kv_rank if self.own_kv else 0))
 
     def cache_needs(self) -> CacheNeeds:
         return CacheNeeds(kv_heads=1, head_dim=self.row, window=self.window or None, values=False)
@@ -109,19 +132,31 @@ class LatentAttention(Mixer):
         ops = self.ops
         ops.set_page_limit(lane.k.shape[0])
         H = self.n_heads
+        if writes_cache != self.own_kv:
+            raise ValueError("latent_attention: a layer with a latent of its own writes its lane, one without reads another's "
+                             "(the schedule and the layer disagree)")
         down = ops.linear(y, self.w_down, out_f32=True)                 # [tokens, q_rank + kv_rank (+ rot_dim) (+ heads)], 32-bit
+        if not self.q_rank:
+            q = ops.latent_prepare(ctx, down, self.g_kv, lane, H, self.d, self.kv_rank, self.rot_dim, self.inv_freq, self.eps,
+                                   write_cache=self.own_kv, adjacent=self.adjacent, magnitude=self.magnitude)
+            return self._attend(ctx, q, lane, None)
         c_q = ops.latent_norm_store(ctx, down, self.g_q, self.g_kv, lane, self.q_rank, self.kv_rank, self.eps, writes_cache,
-                                    rot_dim=self.rot_dim, inv_freq=self.inv_freq, adjacent=self.adjacent)
+                                    rot_dim=self.rot_dim, inv_freq=self.inv_freq, adjacent=self.adjacent, magnitude=self.magnitude)
         if self.rot_dim:
             q = ops.rotate_heads(ctx, ops.linear(c_q, self.w_uq, out_f32=True), H, self.d, self.rot_dim, self.inv_freq,
-                                 self.adjacent)                                          # [tokens, heads * (dim + rot_dim)]
+                                 self.adjacent, self.magnitude)                          # [tokens, heads * (dim + rot_dim)]
         else:
             q = ops.linear(c_q, self.w_uq)                                               # [tokens, heads * dim]
+        return self._attend(ctx, q, lane, down[:, down.shape[1] - H:] if self.gate else None)
+
+    def _attend(self, ctx, q: torch.Tensor, lane, gate: Optional[torch.Tensor]) -> torch.Tensor:
+        """Queries [tokens, heads * (dim (+ rot_dim))] over the lane's rows, through the value map and Wo."""
+        ops, H = self.ops, self.n_heads
         q_lat = ops.head_project(q, self.w_uk, H, out_f32=True)                          # [tokens, heads, row], 32-bit
         # [tokens, heads, row]: 32-bit, unless the map that follows is a library product of many tokens, which takes bf16
         narrow = ops.head_project_by_library(ctx.n_tokens) and ops.latent_attention_on_tensor_cores(self.row)
         o_lat = ops.latent_attention(ctx, q_lat, lane, self.scale, self.window, out_compute_dtype=narrow)
         o = ops.head_project(o_lat, self.w_uv, H, out_f32=False).view(ctx.n_tokens, H * self.vd)
-        if self.gate:
-            ops.head_gate(o, down[:, down.shape[1] - H:], H)
+        if gate is not None:
+            ops.head_gate(o, gate, H)
         return ops.linear(o, self.w_o)

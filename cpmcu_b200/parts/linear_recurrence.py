@@ -13,7 +13,7 @@ from typing import Dict, Optional
 
 import torch
 
-from .base import MIXERS, CacheNeeds, Mixer, WeightSpec
+from .base import MIXERS, POSITIONS, QUERY_TILE_TOKENS, CacheNeeds, Mixer, PartSpec, WeightSpec, build_part
 
 
 class _MatrixStateMixer(Mixer):
@@ -262,3 +262,76 @@ class LightningAttention(_MatrixStateMixer):
         decay = self.decay.unsqueeze(0).expand(ctx.n_tokens, H)             # the same row for every token (stride 0)
         o = ops.linear_recurrence(ctx, q, k, v, decay, None, lane.state["matrix_state"], H, H, d, dv, self.q_scale)
         return ops.linear(ops.gated_group_norm(o, g, self.w_norm, self.eps, self.group, self.gate), self.w_o)
+
+
+@MIXERS.register("retention")
+class Retention(_MatrixStateMixer):
+    """Linear attention with one fixed decay per head and positions by rotation, no softmax and no denominator:
+
+        q = turn(Wq h),  k = turn(Wk h) * d^(-1/2)   (heads x d),   v = Wv h   (heads x dv)
+        S_t = decay_h S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t
+        out = Wo ( o / sqrt(mean(o^2) + eps) * silu(Wg h) )                                      (norm per head, no weight)
+
+    ``position``: the rotation (any magnitude factor it has goes on cosine and sine).  The state [heads, d, dv] is 32-bit per
+    sequence; rotation, decay, recurrence, norm and gate are 32-bit.  A decode step is one kernel between the two products;
+    prompts run by tiles of 64 tokens (what a tile adds to the state, a walk over the tiles' states, the tile's outputs),
+    short portions token by token.  ``names``: "q", "k", "v", "g", "o".
+    """
+
+    DEFAULT_NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o"}
+
+    def __init__(self, ops, hidden_size: int, n_heads: int, head_dim: int, value_dim: int, decay, eps: float,
+                 position: Optional[PartSpec] = None, names=None):
+        super().__init__(ops)
+        self.hidden_size, self.heads, self.d, self.dv, self.eps = int(hidden_size), int(n_heads), int(head_dim), int(value_dim), float(eps)
+        self.decay_values = [float(a) for a in decay]
+        if len(self.decay_values) != self.heads:
+            raise ValueError(f"retention: {self.heads} heads need {self.heads} decays, got {len(self.decay_values)}")
+        if self.d > 256:
+            raise ValueError("retention: the recurrence kernels take heads of up to 256 key channels")
+        enc = build_part(POSITIONS, position if position is not None else PartSpec("none", {}), ops)
+        rot = enc.rotary()
+        if rot is None:
+            raise ValueError("retention takes a rotation of pairs, or no position encoding")
+        self.inv_freq, self.magnitude, self.rot_dim = rot
+        self.adjacent = bool(getattr(enc, "adjacent", False))
+        self.names = dict(self.DEFAULT_NAMES, **(dict(names) if names else {}))
+        self.k_factor = self.d ** -0.5
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        n, W, H, d, dv = self.names, self.hidden_size, self.heads, self.d, self.dv
+        return {n["q"]: WeightSpec((H * d, W)), n["k"]: WeightSpec((H * d, W)), n["v"]: WeightSpec((H * dv, W)),
+                n["g"]: WeightSpec((H * dv, W)), n["o"]: WeightSpec((W, H * dv))}
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        n = self.names
+        self.w_in = self.ops.keep(torch.cat([tensors[n[x]] for x in ("q", "k", "v", "g")], dim=0).contiguous())
+        self.w_o = self.ops.keep(tensors[n["o"]].contiguous())
+        a = torch.tensor(self.decay_values, dtype=torch.float64)
+        powers = a[:, None] ** torch.arange(QUERY_TILE_TOKENS + 1, dtype=torch.float64)[None, :]       # formed once, in 64-bit
+        self.powers = self.ops.keep(powers.float().to(self.w_o.device).contiguous())
+        self.decay = self.ops.keep(a.float().to(self.w_o.device).contiguous())
+
+    def weight_bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_o, self.decay))
+
+    def cache_needs(self) -> CacheNeeds:
+        return CacheNeeds(state={"matrix_state": ((self.heads, self.d, self.dv), torch.float32)})
+
+    def forward(self, ctx, y: torch.Tensor, lane, writes_cache: bool) -> torch.Tensor:
+        ops, H, d, dv = self.ops, self.heads, self.d, self.dv
+        proj = ops.linear(y, self.w_in, out_f32=True)                       # [q | k | v | g]
+        state = lane.state["matrix_state"]
+        if ops.retention_step_ok(ctx, d, dv):
+            o = ops.retention_step(ctx, proj, self.decay, state, H, d, dv, self.inv_freq, self.rot_dim, self.magnitude, self.adjacent,
+                                   self.k_factor, self.eps)
+            return ops.linear(o, self.w_o)
+        ops.rotate_scale(ctx, proj, 2 * H, d, self.inv_freq, self.rot_dim, self.magnitude, self.adjacent, first_scaled=H,
+                         factor=self.k_factor)
+        q, k = proj[:, :H * d], proj[:, H * d:2 * H * d]
+        v, g = proj[:, 2 * H * d:2 * H * d + H * dv], proj[:, 2 * H * d + H * dv:]
+        if ops.retention_tiles_ok(ctx, d, dv):
+            return ops.linear(ops.retention_tiles(ctx, q, k, v, g, self.powers, state, H, d, dv, self.eps), self.w_o)
+        decay = self.decay.unsqueeze(0).expand(ctx.n_tokens, H)             # the same row for every token (stride 0)
+        o = ops.linear_recurrence(ctx, q, k, v, decay, None, state, H, H, d, dv, 1.0)
+        return ops.linear(ops.gated_head_norm(o, g, None, self.eps), self.w_o)

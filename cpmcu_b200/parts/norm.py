@@ -17,14 +17,17 @@ class RMSNorm(Norm):
     recordable_prompt = True
     takes_two_addends = True        # ``add_forward(..., second=)`` adds two deferred outputs in the norm's own pass
 
-    def __init__(self, ops, hidden_size: int, eps: float, weight_name: str = "weight", offset: float = 0.0):
+    def __init__(self, ops, hidden_size: int, eps: float, weight_name: str = "weight", offset: float = 0.0,
+                 wide: bool = False):
         """``weight_name``: the tensor's name below the part's prefix.  ``offset``: a constant added to the stored weight
-        (1 for a weight that is stored around zero: y = x / rms * (1 + w)); the sum is formed once, in 32-bit."""
+        (1 for a weight that is stored around zero: y = x / rms * (1 + w)); the sum is formed once, in 32-bit.  ``wide``: the
+        weight is held in 32-bit whatever it is stored in (``post_forward`` needs it)."""
         super().__init__(ops)
         self.hidden_size = int(hidden_size)
         self.eps = float(eps)
         self.weight_name = str(weight_name)
         self.offset = float(offset)
+        self.wide = bool(wide)
         self.weight: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
@@ -34,6 +37,8 @@ class RMSNorm(Norm):
         w = tensors[self.weight_name]
         if self.offset:
             w = w.float() + self.offset
+        elif self.wide:
+            w = w.float()
         self.weight = self.ops.keep(w.contiguous())
 
     def weight_bytes(self) -> int:
@@ -45,6 +50,11 @@ class RMSNorm(Norm):
     def add_forward(self, x: torch.Tensor, delta: torch.Tensor, scale: float,
                     rows: Optional[torch.Tensor] = None, second: Optional[torch.Tensor] = None) -> torch.Tensor:
         return self.ops.add_rmsnorm(x, delta, scale, self.weight, self.eps, rows, delta2=second)
+
+    def post_forward(self, x: torch.Tensor, a: torch.Tensor, alpha: float, scale: Optional[torch.Tensor]) -> torch.Tensor:
+        """x <- norm(alpha * x + scale * a) in place (``scale``: one fp32 number per channel, or None), the norm after the
+        sum; returns the new x in the compute dtype."""
+        return self.ops.post_norm(x, a, alpha, scale, self.weight, self.eps)
 
 
 @NORMS.register("layer_norm")

@@ -102,6 +102,36 @@ class WavelengthScaledRotary(Rotary):
         self.inv_freq = f.to(torch.float32).to(self.ops.device if self.ops is not None else "cpu")
 
 
+@POSITIONS.register("yarn_rope")
+class YarnRotary(Rotary):
+    """A rotation of the first ``rot_dim`` channels of a head in pairs (i, i + rot_dim/2), f_i = theta^(-2i/rot_dim), with
+    the slow frequencies stretched when ``factor`` is given: with place(t) = rot_dim ln(original / (2 pi t)) / (2 ln theta),
+    the (fractional) i whose wave makes t turns over ``original`` positions, the ramp
+
+        r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1),    lo = max(floor(place(fast)), 0),  hi = min(ceil(place(slow)), rot_dim - 1)
+
+    blends f_i / factor (r = 1) with f_i (r = 0), and cosine and sine are multiplied by 0.1 ln(factor) + 1.  The table is
+    formed in 64-bit on the host and rounded once to 32-bit; angles are 32-bit on the device."""
+
+    def __init__(self, ops, head_dim: int, theta: float, rot_dim: Optional[int] = None, factor: Optional[float] = None,
+                 original: int = 8192, fast: float = 32.0, slow: float = 1.0):
+        super().__init__(ops, head_dim, theta, rot_dim)
+        theta = float(theta)
+        i = torch.arange(self.rot_dim // 2, dtype=torch.float64)
+        f = torch.pow(torch.tensor(theta, dtype=torch.float64), -2.0 * i / max(self.rot_dim, 1))
+        if factor is not None:
+            factor, original, fast, slow = float(factor), float(original), float(fast), float(slow)
+            if not (factor > 0 and original > 0 and fast > 0 and slow > 0 and theta > 0 and theta != 1.0):
+                raise ValueError("yarn_rope: needs positive factor, original, fast and slow, and a base other than 1")
+            place = lambda turns: self.rot_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+            lo = max(math.floor(place(fast)), 0)
+            hi = min(math.ceil(place(slow)), self.rot_dim - 1)
+            ramp = torch.clamp((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+            f = f / factor * ramp + f * (1.0 - ramp)
+            self.magnitude = 0.1 * math.log(factor) + 1.0
+        self.inv_freq = f.to(torch.float32).to(self.ops.device if self.ops is not None else "cpu")
+
+
 @POSITIONS.register("longrope")
 class LongRotary(Rotary):
     def __init__(self, ops, head_dim: int, theta: float, long_factor: Sequence[float],

@@ -122,6 +122,10 @@ def _register_builtin() -> None:
 
     register_architecture(Architecture(name=LukelornConfig.architecture, config_class=LukelornConfig, model_spec=lukelorn.model_spec,
                                        fit_config=lukelorn.fit_config_to_checkpoint))
+    from .config.dinutar import DinutarConfig
+    from .models import dinutar
+
+    register_architecture(Architecture(name=DinutarConfig.architecture, config_class=DinutarConfig, model_spec=dinutar.model_spec))
 
 
 _register_builtin()
