@@ -44,6 +44,9 @@ SEED = 2
 FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
 
 
+FP32_NOMINAL_TFLOPS = 74.4          # 148 SMs x 128 FMA lanes x 2 x 1.965 GHz
+
+
 def long_factors(n: int) -> list:
     import torch
     g = torch.Generator().manual_seed(SEED)
@@ -1505,6 +1508,236 @@ def workload_lukelorn(steps: int, warmup: int, size: str, batch: int) -> int:
     return 0
 
 
+# Dinutar at the sizes of MUFEVIK_SIZES beside Lukelorn at the same sizes (the closest design: attention over a cached latent
+# with a rotated key part, a matrix-state recurrence, a dense feed-forward): eight layers, retention and latent attention
+# in turn, two of the four latent layers reading the rows of the one before them; random weights N(0, 0.02), vectors
+# N(0, 0.02) around one.
+def dinutar_config(z: dict, lat: dict) -> dict:
+    H = z["delta_heads"]
+    mlp = {"kind": "dense", "ff": z["ff"] * z["top"]}
+    ret = {"type": "retention", "mlp": mlp,
+           "mixer": {"heads": H, "dim": z["delta_dim"], "vdim": z["delta_vdim"], "decay": [1.0 - 2.0 ** (-5 - 7 * i / max(1, H - 1)) for i in range(H)],
+                     "rot": {"dims": z["delta_dim"], "base": 10000.0}}}
+
+    def latent(kv_from=None):
+        m = {"heads": z["heads"], "dim": z["dim"], "rot_dim": lat["rot_dim"], "vdim": z["vdim"], "kv_rank": lat["kv_rank"],
+             "scale": (z["dim"] + lat["rot_dim"]) ** -0.5,
+             "rot": {"dims": lat["rot_dim"], "base": 10000.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        if kv_from is not None:
+            m["kv_from"] = kv_from
+        return {"type": "latent_attention", "mlp": mlp, "mixer": m}
+    return {"architecture": "Dinutar", "vocab": z["vocab"], "width": z["width"], "postln_alpha": 2.0, "norm": {"eps": 1e-5},
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}},
+            "layers": [ret, latent(), ret, latent(1), ret, latent(), ret, latent(5)]}
+
+
+def build_dinutar(z: dict, lat: dict, max_tokens: int, max_batch: int, context: int):
+    import torch
+    from cpmcu_b200.engine import Stepper
+    from cpmcu_b200.engine.storage import make_storage
+    from cpmcu_b200.loading import build_model
+    from cpmcu_b200.registry import architecture
+    from cpmcu_b200.weights import random_tensors
+
+    arch = architecture("Dinutar")
+    cfg = arch.config_class.from_dict(dinutar_config(z, lat))
+    model = build_model(arch, cfg, torch.bfloat16, "cuda:0")
+    storage = make_storage(model, PREFILL_TOKENS, max_batch, max_tokens=max_tokens, max_seq_tokens=context + 64, n_slots=max_batch + 2)
+    model.load_weights(random_tensors(model.weight_specs(), 8, torch.bfloat16, std=0.02, norm_mean=1.0, device="cuda:0"))
+    torch.cuda.empty_cache()
+    return cfg, model, storage.cache, Stepper(model, storage.cache, chunk_tokens=PREFILL_TOKENS, graph_prompts=True)
+
+
+def dinutar_kernels(z: dict, lat: dict, pk: dict, context: int, batch: int) -> dict:
+    """Every kernel of the design alone, at the size's shapes, beside the like kernel of the closest models (Lukelorn's
+    latent attention and its preparation, its recurrence with the norm behind it, the fused add + RMS norm, the plain
+    embedding, the gated product): a prompt of 2,048 tokens and a decode step of ``batch`` sequences at ``context``
+    tokens.  CUDA events around one launch (or the launches a row names) after a flush of L2 (a 512 MB buffer is
+    written), median of five; bytes and FLOPs are the algorithmic ones."""
+    import torch
+    from cpmcu_b200.cache import Cache
+    from cpmcu_b200.ops.ops import Ops
+    from cpmcu_b200.parts.base import CacheNeeds, QUERY_TILE_TOKENS, StepContext
+
+    ops = Ops(torch.bfloat16)
+    dev = "cuda:0"
+    flush = torch.empty(512 << 20, dtype=torch.uint8, device=dev)
+    W, H, d, dv, T = z["width"], z["heads"], z["dim"], z["vdim"], PREFILL_TOKENS
+    R, dr, QR = lat["kv_rank"], lat["rot_dim"], lat["q_rank"]
+    RH, rd, rdv, ff, vocab = z["delta_heads"], z["delta_dim"], z["delta_vdim"], z["ff"] * z["top"], z["vocab"]
+    row = R + dr
+    i32 = dict(dtype=torch.int32, device=dev)
+
+    def timed(fn):
+        ts = []
+        for _ in range(6):
+            flush.fill_(1)
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1))
+        return statistics.median(ts[1:])
+
+    def context_of(q_lens, starts, slots):
+        pos = torch.cat([torch.arange(s, s + n) for n, s in zip(q_lens, starts)]).to(**i32)
+        seq = torch.cat([torch.full((n,), i) for i, n in enumerate(q_lens)]).to(**i32)
+        cu = torch.tensor([0] + [sum(q_lens[:i + 1]) for i in range(len(q_lens))], **i32)
+        kv = [s + n for n, s in zip(q_lens, starts)]
+        ctx = StepContext(n_tokens=sum(q_lens), n_seqs=len(q_lens), is_decode=all(n == 1 for n in q_lens), captured=False,
+                          q_lens=list(q_lens), kv_lens=kv, slots=list(slots), max_q_len=max(q_lens), max_kv_len=max(kv),
+                          token_ids=torch.randint(0, vocab, (sum(q_lens),), **i32), positions=pos, token_seq=seq, cu_q=cu,
+                          kv_len_dev=torch.tensor(kv, **i32), slot_dev=torch.tensor(list(slots), **i32))
+        ts = [i for i, n in enumerate(q_lens) for _ in range(0, n, QUERY_TILE_TOKENS)]
+        tr = [r for n in q_lens for r in range(0, n, QUERY_TILE_TOKENS)]
+        ctx.q_tiles = (torch.tensor(ts, **i32), torch.tensor(tr, **i32), len(ts))
+        return ctx
+
+    out = {}
+
+    def note(name, ms, nbytes=0.0, flops=0.0, fp32_flops=0.0, like=None):
+        r = {"us": ms * 1e3}
+        if nbytes:
+            r["gbs"] = nbytes / (ms * 1e-3) / 1e9
+            r["frac_hbm"] = r["gbs"] / pk["hbm_gbs"]
+        if flops:
+            r["tflops"] = flops / (ms * 1e-3) / 1e12
+            r["frac_bf16"] = r["tflops"] / pk["bf16_tflops"]
+        if fp32_flops:                            # work that is 32-bit by the design: beside the nominal FMA rate
+            r["fp32_tflops"] = fp32_flops / (ms * 1e-3) / 1e12
+            r["frac_fp32_nominal"] = r["fp32_tflops"] / FP32_NOMINAL_TFLOPS
+        if like:
+            r["like"] = like
+        out[name] = r
+
+    n_slots = batch + 2
+    cache = Cache([CacheNeeds(kv_heads=1, head_dim=row, values=False)], max_tokens=(batch + 1) * (context + 64), dtype=torch.bfloat16,
+                  device=dev, n_slots=n_slots)
+    slots = [cache.open_sequence() for _ in range(batch)]
+    for s_ in slots:
+        cache.reserve(s_, context)
+    cache.sync()
+    lane = cache.lane(0)
+    lane.k.normal_(0, 0.5)
+    table = torch.randn(vocab, W, device=dev).bfloat16()
+    second = torch.randn(65522, W, device=dev).bfloat16()
+    prev = torch.zeros(n_slots, **i32)
+    w_up = torch.randn(ff, W, device=dev).bfloat16() * 0.02
+    w_gu = torch.randn(2 * ff, W, device=dev).bfloat16() * 0.02
+    wn, ls = torch.ones(W, device=dev), torch.ones(W, device=dev)
+    gkv, gq = torch.ones(R, device=dev), torch.ones(QR, device=dev)
+    inv = torch.ones(max(dr // 2, 1), device=dev)
+    rinv = torch.ones(max(rd // 2, 1), device=dev)
+    decay = torch.full((RH,), 0.99, device=dev)
+    powers = (0.99 ** torch.arange(QUERY_TILE_TOKENS + 1, device=dev, dtype=torch.float32)).repeat(RH, 1).contiguous()
+    state = torch.zeros(n_slots, RH, rd, rdv, device=dev)
+    wv = torch.ones(rdv, device=dev)
+    for phase, q_lens, starts in (("prefill", [T], [0]), ("decode", [1] * batch, [context - 1] * batch)):
+        ctx = context_of(q_lens, starts, slots[:len(q_lens)])
+        n, keys = ctx.n_tokens, [s + j + 1 for nq, s in zip(q_lens, starts) for j in range(nq)]
+        note(f"{phase}/embed_norm (table, pair table, norm)",
+             timed(lambda: ops.embed_norm(ctx, table, 1.0, second, 31, 17, prev, wn, 1e-5)), n * W * 10.0, like="embed_rows (Lukelorn)")
+        note(f"{phase}/embed_rows (Lukelorn)", timed(lambda: ops.embed(ctx.token_ids, table, 1.0)), n * W * 6.0)
+        x, y = torch.randn(n, W, device=dev), torch.randn(n, W, device=dev).bfloat16()
+        note(f"{phase}/post_norm (layer scale, sum, norm; stream and its copy)", timed(lambda: ops.post_norm(x, y, 2.0, ls, wn, 1e-5)),
+             n * W * 12.0, like="add_rmsnorm (one output)")
+        note(f"{phase}/add_rmsnorm (one output)", timed(lambda: ops.add_rmsnorm(x, y, 0.5, wn, 1e-5)), n * W * 12.0)
+        # latent attention: the preparation in one kernel beside Lukelorn's two, the attention without a window beside 1,024
+        cols = H * (d + dr)
+        proj = torch.randn(n, cols + row, device=dev)
+        note(f"{phase}/latent_prepare (queries turned, latent normed and stored)",
+             timed(lambda: ops.latent_prepare(ctx, proj, gkv, lane, H, d, R, dr, inv, 1e-5, magnitude=1.2)), n * (cols + row) * 6.0,
+             like="latent_norm_store + rotate_heads (Lukelorn)")
+        down, qf = torch.randn(n, QR + row, device=dev), torch.randn(n, cols, device=dev)
+
+        def two():
+            ops.latent_norm_store(ctx, down, gq, gkv, lane, QR, R, 1e-5, rot_dim=dr, inv_freq=inv)
+            ops.rotate_heads(ctx, qf, H, d, dr, inv)
+        note(f"{phase}/latent_norm_store + rotate_heads (Lukelorn)", timed(two), n * (cols + QR + row) * 6.0)
+        lane.k.normal_(0, 0.5)
+        q_lat = torch.randn(n, H, row, device=dev)
+        for win, what, like in ((0, "no window", "the same kernel with Lukelorn's window"), (LUKELORN_WINDOW, f"window {LUKELORN_WINDOW}: Lukelorn", None)):
+            seen = [min(k_, win) if win else k_ for k_ in keys]
+            note(f"{phase}/latent_attention (row {row} = rank {R} + rotated {dr}, {what})",
+                 timed(lambda: ops.latent_attention(ctx, q_lat, lane, (d + dr) ** -0.5, win, out_compute_dtype=True)),
+                 nbytes=(sum(seen) * row * 2.0) if phase == "decode" else 0.0, flops=4.0 * H * row * sum(seen), like=like)
+        # retention beside the recurrence of the closest designs with the norm behind it
+        rproj = torch.randn(n, 2 * RH * (rd + rdv), device=dev)
+        q, k = rproj[:, :RH * rd], rproj[:, RH * rd:2 * RH * rd]
+        v, g = rproj[:, 2 * RH * rd:2 * RH * rd + RH * rdv], rproj[:, 2 * RH * rd + RH * rdv:]
+        state_bytes = len(q_lens) * RH * rd * rdv * 8.0
+        io = n * RH * (2.0 * rd + 2.0 * rdv) * 4.0 + n * RH * rdv * 2.0
+        like = "linear_recurrence (delta rule, decay per key channel: Lukelorn) + gated_head_norm"
+        if phase == "prefill":
+            note("prefill/rotate_scale", timed(lambda: ops.rotate_scale(ctx, rproj, 2 * RH, rd, rinv, rd, 1.0, first_scaled=RH, factor=0.1)),
+                 n * RH * rd * 16.0, like="rotate_heads (Lukelorn)")
+            note("prefill/rotate_heads (Lukelorn)", timed(lambda: ops.rotate_heads(ctx, qf, H, d, dr, inv)), n * cols * 6.0)
+            note("prefill/retention_tiles (three kernels; norm and gate in the last)",
+                 timed(lambda: ops.retention_tiles(ctx, q, k, v, g, powers, state, RH, rd, rdv, 1e-5)), nbytes=state_bytes + io,
+                 fp32_flops=2.0 * n * RH * (2 * rd * rdv + QUERY_TILE_TOKENS * (rd + rdv)), like=like)
+        else:
+            note("decode/retention_step (rotation, recurrence, norm and gate)",
+                 timed(lambda: ops.retention_step(ctx, rproj, decay, state, RH, rd, rdv, rinv, rd, 1.0, False, 0.1, 1e-5)),
+                 nbytes=state_bytes + io, like=like)
+        hd = decay.unsqueeze(0).expand(n, RH)
+        note(f"{phase}/linear_recurrence (plain form, one decay per head: Kipizen) + gated_head_norm",
+             timed(lambda: ops.gated_head_norm(ops.linear_recurrence(ctx, q, k, v, hd, None, state, RH, RH, rd, rdv, 1.0), g, wv, 1e-5)),
+             nbytes=state_bytes + io + n * RH * rdv * 8.0, fp32_flops=4.0 * n * RH * rd * rdv)
+        cd, beta = torch.rand(n, RH * rd, device=dev) * 0.1 + 0.9, torch.rand(n, RH, device=dev)
+        note(f"{phase}/linear_recurrence (delta rule, decay per key channel: Lukelorn) + gated_head_norm",
+             timed(lambda: ops.gated_head_norm(ops.linear_recurrence(ctx, q, k, v, cd, beta, state, RH, RH, rd, rdv, 1.0, vector_decay=True), g, wv, 1e-5)),
+             nbytes=state_bytes + io + n * RH * (rd * 4.0 + rdv * 8.0), fp32_flops=6.0 * n * RH * rd * rdv)
+        state.zero_()
+        note(f"{phase}/relu2_linear (up product with relu squared)", timed(lambda: ops.relu2_linear(y, w_up)),
+             nbytes=(ff * W + n * (W + ff)) * 2.0, flops=2.0 * n * ff * W, like="gated_linear (gate and up, SiLU)")
+        note(f"{phase}/gated_linear (gate and up, SiLU)", timed(lambda: ops.gated_linear(y, w_gu, 8)),
+             nbytes=(2 * ff * W + n * (W + ff)) * 2.0, flops=4.0 * n * ff * W)
+    return out
+
+
+def workload_dinutar(steps: int, warmup: int, size: str, batch: int) -> int:
+    """Dinutar at one of MUFEVIK_SIZES beside Lukelorn at the same sizes (the closest design): decode steps of ``batch``
+    sequences ending at a context of 4,096 tokens under a CUDA graph, a prompt of 2,048 tokens, and every kernel of the
+    design alone beside its like."""
+    import torch
+
+    z, lat, pk, context = MUFEVIK_SIZES[size], LUKELORN_LATENT[size], peaks(), CONTEXT
+    cfg, model, cache, stepper = build_dinutar(z, lat, batch * (context + 64) + 128, batch, context)
+    pre_ms = time_prefill_any(stepper, cfg.vocab)
+    ms, clocks, launches, cache_bytes = time_decode(stepper, batch, steps, warmup, cfg.vocab, True, context=context)
+    weight_bytes = model.weight_bytes_per_step()
+    achieved = (weight_bytes + cache_bytes) / (ms * 1e-3) / 1e9
+    del model, cache, stepper
+    torch.cuda.empty_cache()
+    lcfg, lmodel, lcache, lstepper = build_lukelorn(z, lat, batch * (context + 64) + 128, batch, context)
+    l_pre = time_prefill_any(lstepper, lcfg.vocab)
+    l_ms, _, l_launches, l_cache = time_decode(lstepper, batch, steps, warmup, lcfg.vocab, False, context=context)
+    l_weights = lmodel.weight_bytes_per_step()
+    l_achieved = (l_weights + l_cache) / (l_ms * 1e-3) / 1e9
+    del lmodel, lcache, lstepper
+    torch.cuda.empty_cache()
+    kernels = dinutar_kernels(z, lat, pk, context, batch)
+    print(json.dumps({
+        "workload": "dinutar", "metric": f"decode tokens/s (Dinutar {size} sizes, bf16, batch {batch}, context {context})",
+        "value": batch * 1000.0 / ms, "unit": "tokens/s", "ms_per_step": ms, "steps": steps, "warmup": warmup, "dtype": "bf16",
+        "data": "synthetic: uniform-random token ids, random weights N(0,0.02) seed 8",
+        "config": dict({k_: z[k_] for k_ in ("width", "heads", "dim", "vdim", "delta_heads", "delta_dim", "delta_vdim", "vocab")}, **lat,
+                       ff=z["ff"] * z["top"], size=size, layers=len(cfg.layers), global_batch=batch, seq_len=context,
+                       prefill_tokens=PREFILL_TOKENS, cuda_graph=True, peaks=pk["source"]),
+        "prefill": {"value": PREFILL_TOKENS / (pre_ms * 1e-3), "ms": pre_ms},
+        "roofline": {"bound": "hbm", "achieved": achieved, "peak": pk["hbm_gbs"], "unit": "GB/s", "frac": achieved / pk["hbm_gbs"],
+                     "weight_bytes": weight_bytes, "cache_bytes": cache_bytes},
+        "closest_model": {"model": f"Lukelorn at the {size} sizes, {len(lcfg.layers)} layers",
+                          "decode_tokens_s": batch * 1000.0 / l_ms, "ms_per_step": l_ms, "prefill_tokens_s": PREFILL_TOKENS / (l_pre * 1e-3),
+                          "prefill_ms": l_pre, "roofline_frac": l_achieved / pk["hbm_gbs"], "weight_bytes": l_weights,
+                          "cache_bytes": l_cache, "gpu_launches": l_launches},
+        "kernels": kernels, "clocks": clocks, "gpu_launches": launches,
+    }))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1513,13 +1746,15 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=FULL_LAYERS, help="layers built (the full model has 32)")
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--workload", default="dense8b", choices=["dense8b", "half_b", "sparse8b", "reravik", "mufevik", "kipizen", "lukelorn"],
+    ap.add_argument("--workload", default="dense8b", choices=["dense8b", "half_b", "sparse8b", "reravik", "mufevik", "kipizen", "lukelorn",
+                                                                       "dinutar"],
                     help="dense8b: the headline line (8B sizes, batch 8, context 4096); half_b: 0.5B sizes, batch 64, prompts "
                          "uniform in [64, 2048] chunked at 512, decode at context 8192 (256 steps by default); sparse8b: 8B "
                          "sizes with InfLLM-v2, prompts of 16384 and 30000 tokens chunked at 2048, then decode steps; reravik: the Reravik "
                          "design at --size beside MiniCPM4 of equal sizes, and its kernels alone; mufevik: the same for the Mufevik design "
                          "(sizes 1k and 2k); kipizen: the Kipizen design beside Mufevik at the same sizes (1k and 2k), and its kernels alone; "
-                         "lukelorn: the Lukelorn design beside Kipizen at the same sizes (1k and 2k), and its kernels alone")
+                         "lukelorn: the Lukelorn design beside Kipizen at the same sizes (1k and 2k), and its kernels alone; "
+                         "dinutar: the Dinutar design beside Lukelorn at the same sizes (1k and 2k), and its kernels alone")
     ap.add_argument("--size", default="2k", choices=sorted(RERAVIK_SIZES), help="--workload reravik / mufevik: which layer sizes")
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 points and the e2e run")
     ap.add_argument("--kernel", default=None, help="time one kernel alone: skinny_gemm, decode_attention, prefill_attention (tcgen05), prefill_attention_mma, gemm_tcgen05; or run eager steps of a 2-layer model for a launch list: decode_step, prefill_step")
@@ -1557,6 +1792,11 @@ def main() -> int:
             print(f"bench.py: --workload lukelorn takes --size {' or '.join(sorted(MUFEVIK_SIZES))}")
             return 2
         return workload_lukelorn(a.steps, max(3, a.warmup), a.size, a.batch)
+    if a.workload == "dinutar":
+        if a.size not in MUFEVIK_SIZES:
+            print(f"bench.py: --workload dinutar takes --size {' or '.join(sorted(MUFEVIK_SIZES))}")
+            return 2
+        return workload_dinutar(a.steps, max(3, a.warmup), a.size, a.batch)
     if a.kernel:
         return kernel_bench(a.kernel, a.batch, a.ctx, a.rows, a.n, a.k, a.reps)
     a.warmup = max(3, a.warmup)
