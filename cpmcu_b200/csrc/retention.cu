@@ -217,8 +217,10 @@ __device__ __forceinline__ float4 row4(const float* __restrict__ p, int c, int w
     return make_float4(c < width ? p[c] : 0.f, c + 1 < width ? p[c + 1] : 0.f, c + 2 < width ? p[c + 2] : 0.f, c + 3 < width ? p[c + 3] : 0.f);
 }
 
-// A block: 64 key channels x 64 value columns of one tile's U; a thread 4 x 4 of them.
-__global__ void __launch_bounds__(256)
+// A block: 64 key channels x 64 value columns of one tile's U; a thread 8 x 4 of them.
+constexpr int kKvThreads = 128;
+
+__global__ void __launch_bounds__(kKvThreads)
 retention_tile_kv_kernel(const float* __restrict__ k, int64_t k_stride, const float* __restrict__ v, int64_t v_stride,
                          const float* __restrict__ powers /* [heads][65] */, const int* __restrict__ tile_seq,
                          const int* __restrict__ tile_row, const int* __restrict__ cu_q, float* __restrict__ U, int heads, int d, int dv,
@@ -231,9 +233,9 @@ retention_tile_kv_kernel(const float* __restrict__ k, int64_t k_stride, const fl
     const RetTile tl = ret_tile(tile_seq, tile_row, cu_q, blockIdx.x);
     if (tl.n <= 0) return;
     const float* pw = powers + h * (kRetTile + 1);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const int e = threadIdx.x + 256 * i, j = e >> 4, c = 4 * (e & 15);
+#pragma unroll 4
+    for (int e = threadIdx.x; e < kRetTile * 16; e += kKvThreads) {
+        const int j = e >> 4, c = 4 * (e & 15);
         float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), vv = kv;
         if (j < tl.n) {
             kv = row4(k + (int64_t)(tl.t0 + j) * k_stride + (int64_t)h * d, c0 + c, d, vec);
@@ -246,20 +248,20 @@ retention_tile_kv_kernel(const float* __restrict__ k, int64_t k_stride, const fl
     }
     __syncthreads();
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-    float acc[4][4] = {};
-#pragma unroll 8
+    float acc[8][4] = {};
+#pragma unroll 4
     for (int j = 0; j < kRetTile; ++j) {
-        const float4 a = load4(&ks[j][4 * ty]), b = load4(&vs[j][4 * tx]);
-        const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+        const float4 a = load4(&ks[j][8 * ty]), a2 = load4(&ks[j][8 * ty + 4]), b = load4(&vs[j][4 * tx]);
+        const float av[8] = {a.x, a.y, a.z, a.w, a2.x, a2.y, a2.z, a2.w}, bv[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
-        for (int r = 0; r < 4; ++r)
+        for (int r = 0; r < 8; ++r)
 #pragma unroll
             for (int c = 0; c < 4; ++c) acc[r][c] = fmaf(av[r], bv[c], acc[r][c]);
     }
     float* dst = U + ((int64_t)blockIdx.x * heads + h) * d * dv;
 #pragma unroll
-    for (int r = 0; r < 4; ++r) {
-        const int c = c0 + 4 * ty + r, e = e0 + 4 * tx;
+    for (int r = 0; r < 8; ++r) {
+        const int c = c0 + 8 * ty + r, e = e0 + 4 * tx;
         if (c >= d) continue;
         if (vec) {
             if (e < dv) store4(dst + (int64_t)c * dv + e, make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]));
@@ -271,7 +273,7 @@ retention_tile_kv_kernel(const float* __restrict__ k, int64_t k_stride, const fl
     }
 }
 
-constexpr int kScanFlight = 4;       // tiles whose U a thread asks for before it uses the first
+constexpr int kScanFlight = 8;       // tiles whose U a thread asks for at a time, one batch ahead of the one it works on
 
 template <int VEC>
 __global__ void __launch_bounds__(256)
@@ -306,16 +308,20 @@ retention_tile_scan_kernel(float* __restrict__ U, float* __restrict__ state, con
         if (VEC == 4) { const float4 f = load4(st); S[0] = f.x; S[1 % VEC] = f.y; S[2 % VEC] = f.z; S[3 % VEC] = f.w; }
         else S[0] = st[0];
     }
-    for (int i0 = 0; i0 < n_tiles; i0 += kScanFlight) {
-        float u[kScanFlight][VEC];
+    float u[kScanFlight][VEC], next[kScanFlight][VEC];
+    auto fetch = [&](float (&to)[kScanFlight][VEC], int i0) {
 #pragma unroll
         for (int i = 0; i < kScanFlight; ++i) {
             if (i0 + i < n_tiles) {
                 const float* src = u0 + (i0 + i) * step;
-                if (VEC == 4) { const float4 f = load4(src); u[i][0] = f.x; u[i][1 % VEC] = f.y; u[i][2 % VEC] = f.z; u[i][3 % VEC] = f.w; }
-                else u[i][0] = src[0];
+                if (VEC == 4) { const float4 f = load4(src); to[i][0] = f.x; to[i][1 % VEC] = f.y; to[i][2 % VEC] = f.z; to[i][3 % VEC] = f.w; }
+                else to[i][0] = src[0];
             }
         }
+    };
+    fetch(u, 0);
+    for (int i0 = 0; i0 < n_tiles; i0 += kScanFlight) {
+        fetch(next, i0 + kScanFlight);
 #pragma unroll
         for (int i = 0; i < kScanFlight; ++i) {
             if (i0 + i < n_tiles) {
@@ -327,26 +333,34 @@ retention_tile_scan_kernel(float* __restrict__ U, float* __restrict__ state, con
                 for (int j = 0; j < VEC; ++j) S[j] = fmaf(f, S[j], u[i][j]);
             }
         }
+#pragma unroll
+        for (int i = 0; i < kScanFlight; ++i)
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) u[i][j] = next[i][j];
     }
     if (VEC == 4) store4(st, make_float4(S[0], S[1 % VEC], S[2 % VEC], S[3 % VEC]));
     else st[0] = S[0];
 }
 
 // A block: the 64 tokens of a tile x all value columns of a head (NC groups of 64); a thread 4 tokens x 4 NC columns
-// (4 tx + 64 g).  NORM: o / rms(o) * SiLU(gate) in the storage type; else o as it is, fp32 (T = float).
+// (4 tx + 64 g).  One walk over the key channels, a slice at a time, gives the scores of all pairs of the tile and the read-out
+// of the state before it; then the tile's own keys.  NORM: o / rms(o) * SiLU(gate) in the storage type; else o as it is, fp32
+// (T = float).
 template <typename T, int NC, bool NORM>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, NC <= 2 ? 3 : 2)
 retention_tile_out_kernel(const float* __restrict__ q, const float* __restrict__ k, int64_t qk_stride, const float* __restrict__ v,
                           int64_t v_stride, const float* __restrict__ gate, int64_t gate_stride, const float* __restrict__ powers,
                           const int* __restrict__ tile_seq, const int* __restrict__ tile_row, const int* __restrict__ cu_q,
                           const float* __restrict__ S, T* __restrict__ out, int heads, int d, int dv, float eps, int vec) {
-    extern __shared__ __align__(16) float to_smem[];
     constexpr int kCols = 64 * NC;
-    constexpr int kSlice = 32;                    // key channels, keys or state rows that are staged at a time
-    float* qt = to_smem;                          // [d, rounded up to 32][68]: the tile's queries, channel by channel
-    float* as = qt + ((d + 31) & ~31) * kRetPitch;       // [64 keys][68 queries]: decayed scores
-    float* stage = as + kRetTile * kRetPitch;     // [32][max(68, columns)]
+    constexpr int kSlice = NC <= 2 ? 32 : 16;     // key channels, or keys, that are staged at a time
+    __shared__ __align__(16) float qk[kRetTile * kRetPitch];        // a slice of queries and of keys, channel by channel
+    __shared__ __align__(16) float stage[kSlice * kCols];           // rows of the state, or values
     __shared__ float pw[kRetTile + 1];
+    float* qt = qk;
+    float* kt = qk + kSlice * kRetPitch;
+    float* as = qk;                               // later: decayed scores [64 keys][68 queries]
+    static_assert(2 * kSlice <= kRetTile, "the scores take the place of the two slices");
     pdl_launch_dependents();
     pdl_wait();
     const int h = blockIdx.y;
@@ -354,39 +368,59 @@ retention_tile_out_kernel(const float* __restrict__ q, const float* __restrict__
     if (tl.n <= 0) return;
     if (threadIdx.x <= kRetTile) pw[threadIdx.x] = powers[h * (kRetTile + 1) + threadIdx.x];
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const float* qh = q + (int64_t)tl.t0 * qk_stride + (int64_t)h * d;
     const float* kh = k + (int64_t)tl.t0 * qk_stride + (int64_t)h * d;
     const float* vh = v + (int64_t)tl.t0 * v_stride + (int64_t)h * dv;
-    // a warp takes 4 channels of 32 tokens: its stores into the transposed rows hit 32 different banks
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    auto stage_transposed = [&](float* dst, const float* src, int c_first, int c_count) {
-        for (int w = warp; w < 2 * (c_count / 4); w += 8) {
-            const int i = (w & 1) * 32 + lane, c = 4 * (w >> 1);
-            float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (i < tl.n) f = row4(src + (int64_t)i * qk_stride, c_first + c, d, vec);
-            dst[(c + 0) * kRetPitch + i] = f.x;
-            dst[(c + 1) * kRetPitch + i] = f.y;
-            dst[(c + 2) * kRetPitch + i] = f.z;
-            dst[(c + 3) * kRetPitch + i] = f.w;
-        }
-    };
-    stage_transposed(qt, qh, 0, (d + 31) & ~31);
-    // scores of all pairs of the tile
+    const float* Sh = S + ((int64_t)blockIdx.x * heads + h) * d * dv;
     float s[4][4] = {};
+    float o[4][4 * NC] = {};
     for (int c0 = 0; c0 < d; c0 += kSlice) {
+        if (c0) __syncthreads();
+        // a warp takes 4 channels of 32 tokens at a time: its stores into the transposed rows hit 32 different banks
+#pragma unroll
+        for (int u = warp; u < 2 * (kSlice / 4); u += 8) {
+            const int i = (u & 1) * 32 + lane, c = 4 * (u >> 1);
+            float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
+            if (i < tl.n) {
+                a = row4(qh + (int64_t)i * qk_stride, c0 + c, d, vec);
+                b = row4(kh + (int64_t)i * qk_stride, c0 + c, d, vec);
+            }
+            qt[(c + 0) * kRetPitch + i] = a.x;
+            qt[(c + 1) * kRetPitch + i] = a.y;
+            qt[(c + 2) * kRetPitch + i] = a.z;
+            qt[(c + 3) * kRetPitch + i] = a.w;
+            kt[(c + 0) * kRetPitch + i] = b.x;
+            kt[(c + 1) * kRetPitch + i] = b.y;
+            kt[(c + 2) * kRetPitch + i] = b.z;
+            kt[(c + 3) * kRetPitch + i] = b.w;
+        }
+#pragma unroll
+        for (int e = threadIdx.x; e < kSlice * (kCols / 4); e += 256) {
+            const int m = e / (kCols / 4), c = 4 * (e % (kCols / 4));
+            store4(stage + m * kCols + c, c0 + m < d ? row4(Sh + (int64_t)(c0 + m) * dv, c, dv, vec) : make_float4(0.f, 0.f, 0.f, 0.f));
+        }
         __syncthreads();
-        stage_transposed(stage, kh, c0, kSlice);
-        __syncthreads();
-#pragma unroll 8
+#pragma unroll 4
         for (int c = 0; c < kSlice; ++c) {
-            const float4 a = load4(qt + (c0 + c) * kRetPitch + 4 * ty), b = load4(stage + c * kRetPitch + 4 * tx);
+            const float4 a = load4(qt + c * kRetPitch + 4 * ty), b = load4(kt + c * kRetPitch + 4 * tx);
             const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
             for (int r = 0; r < 4; ++r)
 #pragma unroll
                 for (int x = 0; x < 4; ++x) s[r][x] = fmaf(av[r], bv[x], s[r][x]);
+#pragma unroll
+            for (int g = 0; g < NC; ++g) {
+                const float4 z = load4(stage + c * kCols + 64 * g + 4 * tx);
+                const float zv[4] = {z.x, z.y, z.z, z.w};
+#pragma unroll
+                for (int r = 0; r < 4; ++r)
+#pragma unroll
+                    for (int x = 0; x < 4; ++x) o[r][4 * g + x] = fmaf(av[r], zv[x], o[r][4 * g + x]);
+            }
         }
     }
+    __syncthreads();                              // the slices are no longer read: the scores take their place
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
         float w[4];
@@ -396,34 +430,6 @@ retention_tile_out_kernel(const float* __restrict__ q, const float* __restrict__
             w[r] = j <= i ? s[r][x] * pw[i - j] : 0.f;
         }
         store4(as + (4 * tx + x) * kRetPitch + 4 * ty, make_float4(w[0], w[1], w[2], w[3]));
-    }
-    // the state before the tile, read with the queries
-    float o[4][4 * NC] = {};
-    auto product = [&](const float* rows /* [count][68] */, int count) {      // o[i][e] += sum_m rows[m][i] stage[m][e]
-#pragma unroll 4
-        for (int m = 0; m < count; ++m) {
-            const float4 a = load4(rows + m * kRetPitch + 4 * ty);
-            const float av[4] = {a.x, a.y, a.z, a.w};
-#pragma unroll
-            for (int g = 0; g < NC; ++g) {
-                const float4 b = load4(stage + m * kCols + 64 * g + 4 * tx);
-                const float bv[4] = {b.x, b.y, b.z, b.w};
-#pragma unroll
-                for (int r = 0; r < 4; ++r)
-#pragma unroll
-                    for (int x = 0; x < 4; ++x) o[r][4 * g + x] = fmaf(av[r], bv[x], o[r][4 * g + x]);
-            }
-        }
-    };
-    const float* Sh = S + ((int64_t)blockIdx.x * heads + h) * d * dv;
-    for (int c0 = 0; c0 < d; c0 += kSlice) {
-        __syncthreads();
-        for (int e = threadIdx.x; e < kSlice * (kCols / 4); e += 256) {
-            const int m = e / (kCols / 4), c = 4 * (e % (kCols / 4));
-            store4(stage + m * kCols + c, c0 + m < d ? row4(Sh + (int64_t)(c0 + m) * dv, c, dv, vec) : make_float4(0.f, 0.f, 0.f, 0.f));
-        }
-        __syncthreads();
-        product(qt + c0 * kRetPitch, kSlice);
     }
 #pragma unroll
     for (int r = 0; r < 4; ++r) {
@@ -439,7 +445,21 @@ retention_tile_out_kernel(const float* __restrict__ q, const float* __restrict__
             store4(stage + m * kCols + c, j0 + m < tl.n ? row4(vh + (int64_t)(j0 + m) * v_stride, c, dv, vec) : make_float4(0.f, 0.f, 0.f, 0.f));
         }
         __syncthreads();
-        product(as + j0 * kRetPitch, min(kSlice, 8 * warp + 8 - j0));      // a warp's rows end at 8 warp + 7 (count <= 0: none)
+        const int count = min(kSlice, 8 * warp + 8 - j0);                  // a warp's rows end at 8 warp + 7
+#pragma unroll 4
+        for (int m = 0; m < count; ++m) {
+            const float4 a = load4(as + (j0 + m) * kRetPitch + 4 * ty);
+            const float av[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+            for (int g = 0; g < NC; ++g) {
+                const float4 b = load4(stage + m * kCols + 64 * g + 4 * tx);
+                const float bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+                for (int r = 0; r < 4; ++r)
+#pragma unroll
+                    for (int x = 0; x < 4; ++x) o[r][4 * g + x] = fmaf(av[r], bv[x], o[r][4 * g + x]);
+            }
+        }
     }
 #pragma unroll
     for (int r = 0; r < 4; ++r) {
@@ -484,12 +504,8 @@ static int launch_tile_out(const float* q, const float* k, int64_t qk_stride, co
                            int64_t gate_stride, const float* powers, const int* tile_seq, const int* tile_row, int n_tiles,
                            const int* cu_q, const float* S, void* out, int heads, int d, int dv, float eps, int vec,
                            cudaStream_t stream) {
-    const int stage = 64 * NC > kRetPitch ? 64 * NC : kRetPitch;
-    const size_t smem = (size_t)((((d + 31) & ~31) + kRetTile) * kRetPitch + 32 * stage) * sizeof(float);      // at most 120 KiB
     auto kern = retention_tile_out_kernel<T, NC, NORM>;
-    static bool configured[kMaxDevices] = {};
-    if (int e = ensure_dynamic_smem(kern, 128 * 1024, configured)) return e;
-    cpm_launch(kLaunchAttention, kern, dim3(n_tiles, heads), dim3(256), smem, stream, q, k, qk_stride, v, v_stride, gate, gate_stride,
+    cpm_launch(kLaunchAttention, kern, dim3(n_tiles, heads), dim3(256), 0, stream, q, k, qk_stride, v, v_stride, gate, gate_stride,
                powers, tile_seq, tile_row, cu_q, S, (T*)out, heads, d, dv, eps, vec);
     return launch_status();
 }
@@ -509,7 +525,7 @@ CPM_API int cpm_retention_tiles(const float* q, const float* k, int64_t qk_strid
     const int vec = d % 4 == 0 && dv % 4 == 0 && qk_stride % 4 == 0 && v_stride % 4 == 0 && gate_stride % 4 == 0 && aligned(q) && aligned(k) &&
                     aligned(v) && (gate == nullptr || aligned(gate));
     const int c_blocks = (d + 63) / 64, v_blocks = (dv + 63) / 64;
-    cpm_launch(kLaunchAttention, retention_tile_kv_kernel, dim3(n_tiles, heads, c_blocks * v_blocks), dim3(256), 0, stream, k, qk_stride, v,
+    cpm_launch(kLaunchAttention, retention_tile_kv_kernel, dim3(n_tiles, heads, c_blocks * v_blocks), dim3(kKvThreads), 0, stream, k, qk_stride, v,
                v_stride, powers, tile_seq, tile_row, cu_q, scratch, heads, d, dv, v_blocks, vec);
     const int64_t elems = (int64_t)d * dv;
     if (elems % 4 == 0)
