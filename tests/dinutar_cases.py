@@ -73,7 +73,7 @@ def config_b() -> dict:
         _layer(_ret(1, 40, 72, [1.0]), 24),
         _layer(_latent(1, 40, 0, 72, 56, 0.2), 40),
         _layer(_latent(1, 12, 0, 8, 56, 0.5, kv_from=1), 8),
-        _layer(_ret(1, 8, 16, [0.25], rot=(2, 10.0)), None),
+        _layer(_ret(1, 8, 16, [0.9], rot=(2, 10.0)), None),
     ])
 
 
@@ -180,7 +180,7 @@ def random_ids(vocab: int, n: int, seed: int) -> List[int]:
 # bfloat16: activations between the kernels and the cached rows are rounded to bfloat16 in the engine; single rows react
 # strongly to that rounding (a read-out of a retention head is divided by its own size, however small, and squared relus
 # follow), so the worst row has a loose bound and the median a tight one, and float32 carries the exact comparison.
-TOL = {"float32": 6e-5, "bfloat16": 0.3}
+TOL = {"float32": 6e-5, "bfloat16": 0.5}
 MEDIAN_TOL = {"float32": 4e-6, "bfloat16": 1.5e-2}
 
 
