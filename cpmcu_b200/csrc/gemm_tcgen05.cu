@@ -13,8 +13,8 @@
 //
 // Epilogues: bf16 output, or SiLU(gate) * up for a gate_up weight whose rows are interleaved in
 // blocks of 8 (the 32 accumulator columns a thread reads at a time hold 8 gate, 8 up, 8 gate, 8
-// up values of 16 features), or relu(x)^2 (a feed-forward without a gate);
-// each saves the round trip of the intermediate that the reference makes between cublasGemmEx and its activation kernel (src/model/ffn.cuh:38-50).
+// up values of 16 features), or relu(x)^2 (a feed-forward without a gate); each saves the round trip of the
+// intermediate that the reference makes between cublasGemmEx and its activation kernel (src/model/ffn.cuh:38-50).
 //
 // Every wait on a barrier is bounded: when a bound is hit the block records an error code, stops
 // taking work, frees its TMEM and returns, so a fault in the hand-over logic cannot hang the GPU.
